@@ -27,30 +27,12 @@
 #include <cstdlib>
 
 #include "common.cuh"
+#include "decay_exp.cuh"
 
 namespace {
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
-
-// exp(x) for x <= 0, with the last addition the only rounding that counts: a state that decays slowly is multiplied by
-// thousands of such factors in a row, and an error with a sign of its own would add up over a long sequence.
-__device__ __forceinline__ float decay_exp(float x) {
-    if (x < -104.0f) return 0.0f;
-    const float k = rintf(x * 1.442695041f);
-    float r = fmaf(k, -0.693145751953125f, x);
-    r = fmaf(k, -1.428606765330187e-06f, r);
-    float p = 1.9875691500e-4f;
-    p = fmaf(p, r, 1.3981999507e-3f);
-    p = fmaf(p, r, 8.3334519073e-3f);
-    p = fmaf(p, r, 4.1665795894e-2f);
-    p = fmaf(p, r, 1.6666665459e-1f);
-    p = fmaf(p, r, 5.0000001201e-1f);
-    const float e = 1.0f + fmaf(r * r, p, r);
-    const int ki = (int)k;
-    if (ki >= -125) return __int_as_float(__float_as_int(e) + (ki << 23));
-    return __int_as_float(__float_as_int(e) + ((ki + 100) << 23)) * 7.888609052210118e-31f;
-}
 
 constexpr int TILE = 16;        // tokens staged at a time
 constexpr int PAD = 4;          // floats between the parts' rows of a staged key or query: the parts' 16-byte loads then hit different banks
