@@ -29,3 +29,28 @@ EG_API int eg_embedding_gather(cudaStream_t stream, int dtype, const int* ids, c
         embedding_gather_kernel<float><<<tokens, threads, 0, stream>>>(ids, (const float*)table, residual, hidden, vocab, status);
     return eg_launch_status();
 }
+
+// residual[t, 2i] += sin(a), residual[t, 2i + 1] += cos(a) with a = position * f_i, the frequency f_i = head[i] + tail[i] in two float32
+// pieces: the angle's rounding error is worked out and taken into account, so that far positions keep a 32-bit angle.
+namespace {
+__global__ void add_waves_kernel(float* __restrict__ residual, const int* __restrict__ positions, const float* __restrict__ head, const float* __restrict__ tail,
+                                 int tokens, int hidden) {
+    const int pairs = (hidden + 1) / 2;
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long long)tokens * pairs) return;
+    const int t = (int)(i / pairs), c = (int)(i % pairs);
+    const float p = (float)positions[t], f = head[c], a = p * f, rest = fmaf(p, f, -a) + p * tail[c];
+    float s, cs;
+    sincosf(a, &s, &cs);
+    float* x = residual + (size_t)t * hidden + 2 * c;
+    x[0] += fmaf(cs, rest, s);                      // sin(a + rest), rest a few rounding errors of a
+    if (2 * c + 1 < hidden) x[1] += fmaf(-s, rest, cs);
+}
+}  // namespace
+
+EG_API int eg_add_waves(cudaStream_t stream, float* residual, const int* positions, const float* head, const float* tail, int tokens, int hidden) {
+    if (tokens <= 0) return 0;
+    const long long n = (long long)tokens * ((hidden + 1) / 2);
+    add_waves_kernel<<<(unsigned)((n + 127) / 128), 128, 0, stream>>>(residual, positions, head, tail, tokens, hidden);
+    return eg_launch_status();
+}

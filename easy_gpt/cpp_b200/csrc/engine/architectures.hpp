@@ -733,6 +733,105 @@ inline ModelSpec mozalix_spec(const json::Value& config) {
     return spec;
 }
 
+// ---- Zodosun ---------------------------------------------------------------------------------------------------------------
+// A decoder whose config.json lists its layers one by one.  A layer is x = x + mixer(n1(x)), x = x + ff(n2(x)) (or the mixer alone)
+// with RMS norms over norm.groups equal runs of channels; sines and cosines of the position are added to the embedding.  The
+// mixer is one of two: "general_delta" (the delta rule with a decay and a removal rate per head and key channel) and "parallel": an
+// attention whose weights are sigmoids of the scores (biases on q, k and v, a norm over the whole of q and of k, a query temperature
+// that grows with the position, a learned bias by distance, a number per head added to every score, a gate per head) beside a linear
+// attention whose state fades by a constant of the head; the mean of the two outputs, each normed over the width, goes on.  The
+// feed-forward is SwiGLU.  The output is the model's norm, the head and logit_scale.  Every size and constant is a key of
+// config.json, except the rows of the bias tables and the inner size of the decays' maps, which the tensors' shapes give; tensor
+// names are "l<i>.<part>.<tensor>".
+inline ModelSpec zodosun_spec(const json::Value& config) {
+    using C = GufanexConfig;        // the typed readers (a key's path goes into the refusal)
+    if (!config.is_object()) throw ConfigError("config.json is not a JSON object");
+    ModelSpec spec;
+    spec.architecture = "zodosun";
+    const long long width = C::integer(config, "width", ""), vocab = C::integer(config, "vocab", "");
+    if (width <= 0 || vocab <= 0) throw ConfigError("width and vocab must be > 0");
+    const json::Value& norm_keys = C::need(config, "norm", "");
+    const double eps = C::number(norm_keys, "eps", "norm.");
+    const long long groups = C::integer_or(norm_keys, "groups", 1, "norm.");
+    if (eps <= 0.0) throw ConfigError("norm.eps must be > 0");
+    if (groups <= 0 || width % groups) throw ConfigError("norm.groups must divide width");
+    spec.vocab_size = vocab;
+    spec.hidden_size = width;
+    spec.max_positions = C::integer_or(config, "max_positions", 1LL << 30, "");     // the design sets no limit; positions are 32-bit
+    auto norm = [&](const std::string& name) {
+        return PartSpec{"rmsnorm", Params{{"size", width}, {"eps", eps}, {"weight_name", ""}, {"groups", groups}}, name, true};
+    };
+    auto positive = [&](const json::Value& m, const char* key, const std::string& w) {
+        const long long v = C::integer(m, key, w);
+        if (v <= 0) throw ConfigError(w + key + " must be > 0");
+        return v;
+    };
+    const json::Value& layers = C::need(config, "layers", "");
+    if (!layers.is_array() || layers.array.empty()) throw ConfigError("layers must be a list with at least one layer");
+    for (size_t i = 0; i < layers.array.size(); ++i) {
+        const json::Value& l = layers.array[i];
+        const std::string where = "layers[" + std::to_string(i) + "].", prefix = "l" + std::to_string(i), w = where + "mixer.";
+        const json::Value& type = C::need(l, "type", where);
+        const json::Value& m = C::need(l, "mixer", where);
+        if (!type.is_string()) throw ConfigError(where + "type must be a string");
+        PartSpec mixer;
+        if (type.string == "general_delta") {
+            Params d{{"hidden_size", width}, {"heads", positive(m, "heads", w)}, {"dim", positive(m, "dim", w)}, {"eps", eps}, {"unit_eps", 1e-6},
+                     {"decay_scale", std::exp(-0.5)}};
+            if (C::present(m, "rank")) d.set("rank", positive(m, "rank", w));        // only what random-weights mode writes: a file's tensors decide
+            mixer = PartSpec{"general_delta", d, prefix + ".mix", true};
+        } else if (type.string == "parallel") {
+            const json::Value& left = C::need(m, "left", w);
+            const json::Value& right = C::need(m, "right", w);
+            const std::string wl = w + "left.", wr = w + "right.";
+            const long long heads = positive(left, "heads", wl), kv_heads = positive(left, "kv_heads", wl);
+            if (heads % kv_heads) throw ConfigError(wl + "heads must be a multiple of kv_heads");
+            Params a{{"hidden_size", width}, {"heads", heads}, {"kv_heads", kv_heads}, {"dim", positive(left, "dim", wl)}, {"vdim", positive(left, "vdim", wl)},
+                     {"scale", C::number(left, "scale", wl)}, {"norm_eps", eps}, {"bias_max", C::number(left, "bias_max", wl)}, {"distance_bias", 1}, {"head_bias", 1},
+                     {"head_gate", 1}, {"proj_bias", 1}};
+            if (a.real("bias_max") <= 0.0) throw ConfigError(wl + "bias_max must be > 0");
+            if (C::present(left, "q_temp")) {
+                const json::Value& temp = *left.find("q_temp");
+                a.set("temp_coef", C::number(temp, "coef", wl + "q_temp."));
+                a.set("temp_every", positive(temp, "every", wl + "q_temp."));
+            }
+            const long long fading = positive(right, "heads", wr);
+            Params r{{"hidden_size", width}, {"heads", fading}, {"dim", positive(right, "dim", wr)}, {"vdim", positive(right, "vdim", wr)}, {"eps", eps}};
+            const json::Value& decay = C::need(right, "decay", wr);
+            if (!decay.is_array() || (long long)decay.array.size() != fading) throw ConfigError(wr + "decay must list one number per head");
+            for (long long h = 0; h < fading; ++h) {
+                if (!decay.array[h].is_number()) throw ConfigError(wr + "decay must list one number per head");
+                r.set("decay." + std::to_string(h), decay.array[h].number);
+            }
+            Params both{{"left_kind", "sigmoid_attention"}, {"right_kind", "lightning"}, {"hidden_size", width}, {"norm_eps", eps}, {"norm_scale", 0.5}};
+            both.merge("left.", a);
+            both.merge("right.", r);
+            mixer = PartSpec{"side_by_side", both, prefix + ".mix", true};
+        } else {
+            throw ConfigError(where + "type '" + type.string + "' is no mixer of this design (parallel, general_delta)");
+        }
+        LayerSpec layer;
+        layer.sublayers.push_back({"mixer", mixer, norm(prefix + ".norm1"), "pre", PartSpec::none()});
+        if (C::present(l, "mlp")) {
+            const json::Value& mlp = *l.find("mlp");
+            const std::string wm = where + "mlp.";
+            const json::Value& kind = C::need(mlp, "kind", wm);
+            if (!kind.is_string() || kind.string != "dense") throw ConfigError(wm + "kind must be 'dense'");
+            Params f{{"hidden_size", width}, {"intermediate_size", positive(mlp, "ff", wm)}, {"gate_name", ".gate"}, {"up_name", ".up"}, {"down_name", ".down"}};
+            layer.sublayers.push_back({"feed_forward", PartSpec{"swiglu", f, prefix + ".mlp", true}, norm(prefix + ".norm2"), "pre", PartSpec::none()});
+        }
+        spec.layers.push_back(std::move(layer));
+        spec.run_order.push_back(RunEntry{(int)i, (int)i, true});
+    }
+    spec.embedding = PartSpec{"embedding", Params{{"vocab_size", vocab}, {"hidden_size", width}, {"weight_name", ""}}, "embed", true};
+    spec.embedding_position = PartSpec{"waves", Params{{"size", width}, {"base", 10000.0}}, "", true};
+    spec.final_norm = norm("final.norm");
+    Params head{{"vocab_size", vocab}, {"hidden_size", width}, {"weight_name", ""}};
+    if (C::present(config, "logit_scale")) head.set("scale", C::number(config, "logit_scale", ""));
+    spec.lm_head = PartSpec{"lm_head", head, "head", true};
+    return spec;
+}
+
 inline void register_builtin_architectures() {
     ArchitectureRegistry& r = ArchitectureRegistry::instance();
     for (auto& e : r.entries)
@@ -742,6 +841,7 @@ inline void register_builtin_architectures() {
     r.add("lasizen", lasizen_spec);
     r.add("masezen", masezen_spec);
     r.add("mozalix", mozalix_spec);
+    r.add("zodosun", zodosun_spec);
 }
 
 }  // namespace easygpt::engine

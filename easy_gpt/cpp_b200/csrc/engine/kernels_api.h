@@ -183,4 +183,26 @@ int eg_gemm_tcgen05_pair_glu_bias(cudaStream_t stream, const void* A, long long 
 int eg_rmsnorm_add_rows(cudaStream_t stream, float* residual, const void* y, int y_dtype, long long ldy, const float* bias, const float* gain, float eps, void* out, int out_dtype, int tokens, int hidden);
 // attention_tcgen05.cu
 int eg_attention_prefill_tcgen05_masked(cudaStream_t stream, const void* q, long long ldq, int total_tokens, const void* k_cache, const void* v_cache, const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, void* out, int out_dtype, long long ldo, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale, const float* sinks, float out_scale, int* status, int max_parts, int part_tiles, float* partial_o, float* partial_ml, int* queue);
+// norm.cu
+int eg_add_group_rmsnorm(cudaStream_t stream, int delta_dtype, int out_dtype, float* residual, const void* delta, const int* rows, const float* gain, void* out, int num_rows, int hidden, int groups, float eps);
+// embedding.cu
+int eg_add_waves(cudaStream_t stream, float* residual, const int* positions, const float* head, const float* tail, int tokens, int hidden);
+// sandwich.cu
+int eg_rmsnorm_pair(cudaStream_t stream, const float* a, const float* b, const float* gain_a, const float* gain_b, float eps, float factor, float* out, int tokens, int hidden);
+// attention_sigmoid.cu
+int eg_sigmoid_attention_prepare(cudaStream_t stream, int dtype, const float* proj, long long ld, const float* bias, const float* q_gain, const float* k_gain, float eps, float temp_coef, int temp_every, const int* positions, const int* slot_map, void* k_cache, void* v_cache, int row_stride, long long head_stride, int page_size, long long page_stride, long long pool_slots, void* q_out, int tokens, int heads, int kv_heads, int dk, int dv, int* status);
+// attention_sigmoid.cu
+int eg_sigmoid_attention(cudaStream_t stream, int dtype, const void* q, const void* k_cache, const void* v_cache, int row_stride, long long head_stride, const int* block_table, int table_stride, const int* token_seq, const int* positions, const float* bias_table, int reach, const float* gate, long long ld_gate, void* out, long long ldo, int tokens, int heads, int kv_heads, int dk, int dv, int page_size, long long page_stride, int num_pages, float scale, int* status);
+// attention_sigmoid.cu
+int eg_sigmoid_attention_mma_takes(int dk, int dv, int reach);
+// attention_sigmoid.cu
+int eg_sigmoid_attention_tiles(cudaStream_t stream, const void* q, const void* k_cache, const void* v_cache, int row_stride, long long head_stride, const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, const float* bias_table, int reach, const float* gate, long long ld_gate, void* out, long long ldo, int heads, int kv_heads, int dk, int dv, int page_size, long long page_stride, int num_pages, float scale, int* status);
+// attention_sigmoid.cu
+int eg_sigmoid_attention_split(cudaStream_t stream, const void* q, const void* k_cache, const void* v_cache, int row_stride, long long head_stride, const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* token_list, int num_tokens, const float* bias_table, int reach, const float* gate, long long ld_gate, void* out, long long ldo, float* partial, int* counters, int splits, int heads, int kv_heads, int dk, int dv, int page_size, long long page_stride, int num_pages, float scale, int* status);
+// general_delta.cu
+int eg_general_delta(cudaStream_t stream, const float* proj, long long ldp, int r_col, int k_col, int v_col, int g_col, int a_col, const float* x, long long ldx, const float* w0, const float* a0, const float* gain, float* vecs, float* state, long long slot_floats, long long state_offset, const int* seq_starts, const int* seq_slots, void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps, float eps, float decay_scale);
+// general_delta.cu
+int eg_tanh_columns(cudaStream_t stream, const float* src, long long lds, void* dst, int dst_dtype, long long ldd, int rows, int cols, int padded);
+// lightning.cu
+int eg_lightning(cudaStream_t stream, const float* proj, long long ldp, int q_col, int k_col, int v_col, int g_col, const float* decays, const float* gain, float* state, long long slot_floats, long long state_offset, const int* seq_starts, const int* seq_slots, float* o_raw, void* y, int y_dtype, long long ldy, int slices, int tokens, int num_seqs, int heads, int dk, int dv, float eps);
 }  // extern "C"

@@ -11,6 +11,7 @@
 #include "parts_masked.hpp"
 #include "parts_mixed.hpp"
 #include "parts_sequence.hpp"
+#include "parts_sigmoid.hpp"
 
 namespace easygpt::engine {
 
@@ -359,6 +360,7 @@ public:
         register_delta_parts();
         register_mixed_parts();
         register_masked_parts();
+        register_sigmoid_parts();
         spec.validate();
         PartRegistry& reg = PartRegistry::instance();
         embedding = PartRegistry::find(reg.embeddings, "embedding", spec.embedding.kind)(spec.embedding.params, spec.embedding.prefix);

@@ -253,12 +253,15 @@ private:
 };
 
 // ---- RMSNorm: y = w * (x / sqrt(mean(x^2) + eps)) (src/models/norm.cpp:46-60), eps a parameter (the reference fixes
-// 1e-6, src/models/norm.cpp:41), fused with the float32 residual add; with single_gain the stored gain is one number ---------------------------------------------------
+// 1e-6, src/models/norm.cpp:41), fused with the float32 residual add; with single_gain the stored gain is one number; with
+// groups the row is cut into that many equal runs of channels, each over its own root mean square ------------------------
 class RMSNorm : public Norm {
 public:
     RMSNorm(const Params& p, const std::string& prefix)
         : Norm(p, prefix), size_((int)p.integer("size")), eps_((float)p.real("eps")), weight_name_(prefix + p.text("weight_name", ".weight")),
-          single_(p.integer("single_gain", 0) != 0), offset_((float)p.real("offset", 0.0)) {}
+          single_(p.integer("single_gain", 0) != 0), offset_((float)p.real("offset", 0.0)), groups_((int)p.integer("groups", 1)) {
+        if (groups_ < 1 || size_ % groups_) throw std::invalid_argument("a norm's size must be a multiple of its groups");
+    }
     std::vector<TensorRequest> tensor_requests() const override {
         return {(single_ ? TensorRequest::scalar(weight_name_) : TensorRequest::vector(weight_name_, size_)).with_init(offset_ != 0.f ? "zero" : "one")};
     }
@@ -272,21 +275,29 @@ public:
     size_t weight_bytes() const override { return (size_t)size_ * 4; }
     bool capturable() const override { return true; }
     bool rms_parameters(const float** gain, float* eps) const override {
+        if (groups_ > 1) return false;             // the kernels that fold a norm in know one root mean square a row
         *gain = gain_.as<float>();
         *eps = eps_;
         return true;
     }
     void forward(const StepContext& ctx, float* residual, const void* delta, DType delta_dtype, void* out, DType out_dtype, int num_rows,
                  const int* rows) const override {
+        if (groups_ > 1) {
+            launch_check(eg_add_group_rmsnorm(ctx.stream, (int)(delta ? delta_dtype : out_dtype), (int)out_dtype, residual, delta, rows, gain_.as<float>(), out,
+                                              num_rows, size_, groups_, eps_), "add_group_rmsnorm");
+            return;
+        }
         launch_check(eg_add_rmsnorm(ctx.stream, (int)(delta ? delta_dtype : out_dtype), (int)out_dtype, residual, delta, rows, gain_.as<float>(), out,
                                     num_rows, size_, eps_), "add_rmsnorm");
     }
     bool add_normed(const StepContext& ctx, float* residual, const void* y, DType y_dtype, int num_rows) const override {
+        if (groups_ > 1) return false;
         launch_check(eg_rmsnorm_add(ctx.stream, residual, y, (int)y_dtype, size_, gain_.as<float>(), eps_, num_rows, size_), "rmsnorm_add");
         return true;
     }
     bool add_normed_rows(const StepContext& ctx, float* residual, const void* y, DType y_dtype, const float* bias, int num_rows, void* out,
                          DType out_dtype) const override {
+        if (groups_ > 1) return false;
         const int rc = eg_rmsnorm_add_rows(ctx.stream, residual, y, (int)y_dtype, size_, bias, gain_.as<float>(), eps_, out, (int)out_dtype, num_rows, size_);
         if (rc == (int)cudaErrorInvalidValue) return false;      // a size the fused kernel does not take
         launch_check(rc, "rmsnorm_add_rows");
@@ -296,7 +307,7 @@ public:
                          DType out_dtype) const override {
         const float* gain2 = nullptr;
         float eps2 = 0.f;
-        if (!next || next->size() != size_ || !next->rms_parameters(&gain2, &eps2)) return false;
+        if (groups_ > 1 || !next || next->size() != size_ || !next->rms_parameters(&gain2, &eps2)) return false;
         const int rc = eg_rmsnorm_add_norm(ctx.stream, residual, y, (int)y_dtype, size_, gain_.as<float>(), eps_, gain2, eps2, out, (int)out_dtype, num_rows, size_);
         if (rc == (int)cudaErrorInvalidValue) return false;      // a size the fused kernel does not take
         launch_check(rc, "rmsnorm_add_norm");
@@ -310,6 +321,7 @@ private:
     std::string weight_name_;      // parameter weight_name: the gain's tensor name as a suffix of the prefix (default ".weight")
     bool single_;                  // parameter single_gain: the tensor is ONE number, the gain of every coordinate
     float offset_;                 // parameter offset: the gain is offset + the stored tensor (1 where the file holds the gain minus one)
+    int groups_;                   // parameter groups: equal runs of channels, each over its own root mean square (default 1)
     DeviceBuffer gain_;
 };
 

@@ -353,9 +353,11 @@ private:
 
 // ---- two mixers side by side --------------------------------------------------------------------------------------------------
 // out = left(h) + right(h): both read the same rows; their weights on the sum are parameters of the two mixers themselves
-// (out_scale), so the sum costs one addition.  The two are built from the registry by kind; the first may keep pages, the
+// (out_scale), so the sum costs one addition.  With norm_eps given, each output is first divided by its root mean square over the
+// width (norm_eps under the root) and multiplied by a gain per channel (tensors .left.out and .right.out), and the sum carries
+// the factor norm_scale: one kernel.  The two are built from the registry by kind; the first may keep pages, the
 // second a state (or either nothing): the cache manager gives the pair pages AND a slot.
-// Parameters: left_kind, right_kind, and the two mixers' own parameters under "left." and "right.".  Tensors: the two mixers'
+// Parameters: left_kind, right_kind, hidden_size with norm_eps and norm_scale, and the two mixers' own parameters under "left." and "right.".  Tensors: the two mixers'
 // under <prefix>.left and <prefix>.right.
 class SideBySideMixer : public Mixer {
 public:
@@ -363,11 +365,17 @@ public:
     std::vector<TensorRequest> tensor_requests() const override {
         std::vector<TensorRequest> r = left_->tensor_requests();
         for (auto& t : right_->tensor_requests()) r.push_back(t);
+        if (norm_eps_ > 0.f)
+            for (const char* n : {".left.out", ".right.out"}) r.push_back(TensorRequest::vector(prefix + n, hidden_).with_init("one"));
         return r;
     }
     void load(const HostTensors& file, DType dtype) override {
         left_->load(file, dtype);
         right_->load(file, dtype);
+        if (norm_eps_ > 0.f) {
+            left_gain_ = upload_f32(file, prefix + ".left.out");
+            right_gain_ = upload_f32(file, prefix + ".right.out");
+        }
     }
     size_t weight_bytes() const override { return left_->weight_bytes() + right_->weight_bytes(); }
     size_t arena_bytes(long long T) const override { return left_->arena_bytes(T) + right_->arena_bytes(T); }
@@ -393,16 +401,27 @@ public:
         Delta a = left_->forward(ctx, rows, left_paged ? paged : slot, nullptr);
         Delta b = right_->forward(ctx, rows, left_paged ? slot : paged, nullptr);
         if (a.has_pre() || b.has_pre() || a.scale || b.scale || a.dtype != DType::F32) throw DeviceError("two mixers side by side hand back plain float32 outputs");
+        if (norm_eps_ > 0.f) {
+            if (b.dtype != DType::F32) throw DeviceError("two mixers side by side hand back plain float32 outputs");
+            launch_check(eg_rmsnorm_pair(ctx.stream, (const float*)a.p, (const float*)b.p, left_gain_.as<float>(), right_gain_.as<float>(), norm_eps_, norm_scale_,
+                                         (float*)a.p, ctx.num_tokens, hidden_), "rmsnorm_pair");
+            return a;
+        }
         launch_check(eg_add_into_f32(ctx.stream, (float*)a.p, b.p, (int)b.dtype, (long long)ctx.num_tokens * h.cols), "add");
         return a;
     }
 
 private:
     std::shared_ptr<Mixer> left_, right_;
+    int hidden_;
+    float norm_eps_, norm_scale_;
+    DeviceBuffer left_gain_, right_gain_;
 };
 
 inline SideBySideMixer::SideBySideMixer(const Params& p, const std::string& prefix, std::shared_ptr<PositionEncoding> position)
-    : Mixer(p, prefix, position) {
+    : Mixer(p, prefix, position), hidden_((int)p.integer("hidden_size", 0)), norm_eps_((float)p.real("norm_eps", 0.0)),
+      norm_scale_((float)p.real("norm_scale", 1.0)) {
+    if (norm_eps_ > 0.f && hidden_ <= 0) throw std::invalid_argument("two mixers side by side: norms on their outputs need hidden_size");
     PartRegistry& reg = PartRegistry::instance();
     left_ = PartRegistry::find(reg.mixers, "mixer", p.text("left_kind"))(p.sub("left."), prefix + ".left", position);
     right_ = PartRegistry::find(reg.mixers, "mixer", p.text("right_kind"))(p.sub("right."), prefix + ".right", position);

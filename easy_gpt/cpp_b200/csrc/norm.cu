@@ -6,15 +6,26 @@
 // correctly rounded (no fast-math).  With `rows` given, output row r is computed
 // from residual row rows[r] (the final norm runs only where logits are wanted)
 // and the residual is left untouched.
+//
+// With groups > 1 every row is cut into that many equal runs of channels, each normalised by its own root mean square (the gain is
+// one per channel as before): a run is treated as a row of its own, `part` channels long.
 #include "common.cuh"
 
-template <typename TD, typename TO>
+// the row of the residual that output run r (of row r / groups) is computed from, as a run index
+template <bool GROUPED>
+__device__ __forceinline__ int source_run(const int* __restrict__ rows, int r, int groups) {
+    if (!GROUPED) return rows ? rows[r] : r;
+    return rows ? rows[r / groups] * groups + r % groups : r;
+}
+
+template <typename TD, typename TO, bool GROUPED>
 __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TD* __restrict__ delta,
                                    const int* __restrict__ rows, const float* __restrict__ gain,
-                                   TO* __restrict__ out, int hidden, float eps) {
+                                   TO* __restrict__ out, int hidden, float eps, int groups) {
     __shared__ float scratch[32];
     const int r = blockIdx.x;
-    const int src = rows ? rows[r] : r;
+    const int src = source_run<GROUPED>(rows, r, groups);
+    if (GROUPED) gain += (r % groups) * hidden;
     float* x = residual + (size_t)src * hidden;
     const TD* d = delta ? delta + (size_t)src * hidden : nullptr;
     const bool write_back = (rows == nullptr) && (d != nullptr);
@@ -40,14 +51,15 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TD* __res
 // the row is read once, all of its loads are in flight at once, the sum is a shuffle, and nothing waits at a barrier.
 // (Measured on B200, 2,048 rows of 896: 5.6 us a launch with a block per row and a sum through shared memory.)
 // The sum's order (a lane's values in order, then the lanes by halving) depends on the width alone.
-template <typename TD, typename TO, int VPL>
+template <typename TD, typename TO, int VPL, bool GROUPED>
 __global__ void __launch_bounds__(256) add_rmsnorm_warp_kernel(float* __restrict__ residual, const TD* __restrict__ delta,
                                                                const int* __restrict__ rows, const float* __restrict__ gain,
-                                                               TO* __restrict__ out, int num_rows, int hidden, float eps) {
+                                                               TO* __restrict__ out, int num_rows, int hidden, float eps, int groups) {
     const int lane = threadIdx.x & 31;
     const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (r >= num_rows) return;
-    const int src = rows ? rows[r] : r;
+    const int src = source_run<GROUPED>(rows, r, groups);
+    if (GROUPED) gain += (r % groups) * hidden;
     const int quads = hidden / 4;
     float4* x = reinterpret_cast<float4*>(residual + (size_t)src * hidden);
     float4 v[VPL];
@@ -114,42 +126,60 @@ __global__ void __launch_bounds__(256) add_rmsnorm_warp_kernel(float* __restrict
     }
 }
 
-template <typename TD, typename TO>
+template <typename TD, typename TO, bool GROUPED>
 static void launch_warp_norm(cudaStream_t stream, float* residual, const void* delta, const int* rows, const float* gain, void* out, int num_rows,
-                             int hidden, float eps) {
+                             int hidden, float eps, int groups) {
     const int vpl = (hidden / 4 + 31) / 32;
     // few rows: a warp a block, so that they are spread over the SMs (64 rows: 1.72 ms a decode step with eight warps a
     // block, 1.58 with one)
     const int warps = num_rows >= 2048 ? 8 : num_rows >= 512 ? 2 : 1, blocks = (num_rows + warps - 1) / warps;
 #define EG_WARP_NORM(V) \
-    add_rmsnorm_warp_kernel<TD, TO, V><<<blocks, warps * 32, 0, stream>>>(residual, (const TD*)delta, rows, gain, (TO*)out, num_rows, hidden, eps)
-    if (vpl <= 4) EG_WARP_NORM(4);
+    add_rmsnorm_warp_kernel<TD, TO, V, GROUPED><<<blocks, warps * 32, 0, stream>>>(residual, (const TD*)delta, rows, gain, (TO*)out, num_rows, hidden, eps, groups)
+    if (GROUPED && vpl <= 1) EG_WARP_NORM(1);
+    else if (vpl <= 4) EG_WARP_NORM(4);
     else if (vpl <= 8) EG_WARP_NORM(8);
     else if (vpl <= 16) EG_WARP_NORM(16);
     else EG_WARP_NORM(32);
 #undef EG_WARP_NORM
 }
 
-// delta_dtype / out_dtype: EG_F32 or EG_BF16.  rows may be null.  delta may be null.
-EG_API int eg_add_rmsnorm(cudaStream_t stream, int delta_dtype, int out_dtype, float* residual, const void* delta,
-                          const int* rows, const float* gain, void* out, int num_rows, int hidden, float eps) {
-    if (num_rows <= 0) return 0;
+// num_rows runs of `hidden` channels (GROUPED: `groups` runs a row)
+template <bool GROUPED>
+static int launch_norm(cudaStream_t stream, int delta_dtype, int out_dtype, float* residual, const void* delta, const int* rows, const float* gain, void* out,
+                       int num_rows, int hidden, float eps, int groups) {
     if (hidden % 4 == 0 && hidden <= 4096 && (uintptr_t)residual % 16 == 0 && (uintptr_t)gain % 16 == 0 &&
         (uintptr_t)out % 16 == 0 && (!delta || (uintptr_t)delta % 16 == 0)) {
-        if (delta_dtype == EG_BF16 && out_dtype == EG_BF16) launch_warp_norm<bf16, bf16>(stream, residual, delta, rows, gain, out, num_rows, hidden, eps);
-        else if (delta_dtype == EG_F32 && out_dtype == EG_F32) launch_warp_norm<float, float>(stream, residual, delta, rows, gain, out, num_rows, hidden, eps);
-        else if (delta_dtype == EG_BF16 && out_dtype == EG_F32) launch_warp_norm<bf16, float>(stream, residual, delta, rows, gain, out, num_rows, hidden, eps);
-        else launch_warp_norm<float, bf16>(stream, residual, delta, rows, gain, out, num_rows, hidden, eps);
+#define EG_NORM_LAUNCH(TD, TO) launch_warp_norm<TD, TO, GROUPED>(stream, residual, delta, rows, gain, out, num_rows, hidden, eps, groups)
+        if (delta_dtype == EG_BF16 && out_dtype == EG_BF16) EG_NORM_LAUNCH(bf16, bf16);
+        else if (delta_dtype == EG_F32 && out_dtype == EG_F32) EG_NORM_LAUNCH(float, float);
+        else if (delta_dtype == EG_BF16 && out_dtype == EG_F32) EG_NORM_LAUNCH(bf16, float);
+        else EG_NORM_LAUNCH(float, bf16);
+#undef EG_NORM_LAUNCH
         return eg_launch_status();
     }
     int threads = 128;
     while (threads < 1024 && threads * 4 < hidden) threads <<= 1;
 #define EG_NORM_LAUNCH(TD, TO) \
-    add_rmsnorm_kernel<TD, TO><<<num_rows, threads, 0, stream>>>(residual, (const TD*)delta, rows, gain, (TO*)out, hidden, eps)
+    add_rmsnorm_kernel<TD, TO, GROUPED><<<num_rows, threads, 0, stream>>>(residual, (const TD*)delta, rows, gain, (TO*)out, hidden, eps, groups)
     if (delta_dtype == EG_BF16 && out_dtype == EG_BF16) EG_NORM_LAUNCH(bf16, bf16);
     else if (delta_dtype == EG_F32 && out_dtype == EG_F32) EG_NORM_LAUNCH(float, float);
     else if (delta_dtype == EG_BF16 && out_dtype == EG_F32) EG_NORM_LAUNCH(bf16, float);
     else EG_NORM_LAUNCH(float, bf16);
 #undef EG_NORM_LAUNCH
     return eg_launch_status();
+}
+
+// delta_dtype / out_dtype: EG_F32 or EG_BF16.  rows may be null.  delta may be null.
+EG_API int eg_add_rmsnorm(cudaStream_t stream, int delta_dtype, int out_dtype, float* residual, const void* delta,
+                          const int* rows, const float* gain, void* out, int num_rows, int hidden, float eps) {
+    if (num_rows <= 0) return 0;
+    return launch_norm<false>(stream, delta_dtype, out_dtype, residual, delta, rows, gain, out, num_rows, hidden, eps, 1);
+}
+
+// The same with every row cut into `groups` equal runs of channels (hidden a multiple of groups), each over its own root mean square.
+EG_API int eg_add_group_rmsnorm(cudaStream_t stream, int delta_dtype, int out_dtype, float* residual, const void* delta, const int* rows, const float* gain,
+                                void* out, int num_rows, int hidden, int groups, float eps) {
+    if (num_rows <= 0) return 0;
+    if (groups <= 0 || hidden % groups) return (int)cudaErrorInvalidValue;
+    return launch_norm<true>(stream, delta_dtype, out_dtype, residual, delta, rows, gain, out, num_rows * groups, hidden / groups, eps, groups);
 }

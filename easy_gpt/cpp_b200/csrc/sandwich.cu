@@ -4,6 +4,7 @@
 //                                                                    slot holds the last row of earlier steps (zeros at the start)
 //   norm + shift     the same with h = gain * x / sqrt(mean(x^2) + eps) computed here from the float32 stream
 //   norm and add     x[t] += gain * y[t] / sqrt(mean(y[t]^2) + eps)  a branch's output joins the stream through its norm
+//   two branches     out[t] = factor * (gain_a a[t] / rms(a[t]) + gain_b b[t] / rms(b[t]))   two mixers side by side, each normed
 //   xIELU            a(z) = ap z^2 + z / 2 (z > 0),  an (e^z - 1 - z) + z / 2 (z <= 0)
 //   scaled gather    x[t] = scale * table[id[t]]
 //
@@ -276,6 +277,45 @@ __global__ void __launch_bounds__(256) rmsnorm_shift_warp_kernel(const float* __
     }
 }
 
+// out may be a; a and b float32, a warp per row with both rows in registers
+template <int VPL>
+__global__ void __launch_bounds__(256) rmsnorm_pair_warp_kernel(const float* a, const float* __restrict__ b, const float* __restrict__ gain_a,
+                                                                const float* __restrict__ gain_b, float eps, float factor, float* out, int tokens, int hidden) {
+    const int lane = threadIdx.x & 31, t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (t >= tokens) return;
+    const int quads = hidden / 4;
+    float4 u[VPL], v[VPL];
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+        const int q = i * 32 + lane;
+        u[i] = q < quads ? load4(a + (size_t)t * hidden, q) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[i] = q < quads ? load4(b + (size_t)t * hidden, q) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    float sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+        sa += squares(u[i]);
+        sb += squares(v[i]);
+    }
+    const float fa = factor / sqrtf(warp_sum(sa) / (float)hidden + eps), fb = factor / sqrtf(warp_sum(sb) / (float)hidden + eps);
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+        const int q = i * 32 + lane;
+        if (q >= quads) continue;
+        const float4 g = load4(gain_a, q), h = load4(gain_b, q);
+        store4(out + (size_t)t * hidden, q, make_float4(fmaf(h.x, v[i].x * fb, g.x * (u[i].x * fa)), fmaf(h.y, v[i].y * fb, g.y * (u[i].y * fa)),
+                                                        fmaf(h.z, v[i].z * fb, g.z * (u[i].z * fa)), fmaf(h.w, v[i].w * fb, g.w * (u[i].w * fa))));
+    }
+}
+__global__ void rmsnorm_pair_kernel(const float* a, const float* __restrict__ b, const float* __restrict__ gain_a, const float* __restrict__ gain_b, float eps,
+                                    float factor, float* out, int hidden) {
+    __shared__ float scratch[32];
+    const float *x = a + (size_t)blockIdx.x * hidden, *y = b + (size_t)blockIdx.x * hidden;
+    const float fa = factor * inv_rms(x, hidden, eps, scratch), fb = factor * inv_rms(y, hidden, eps, scratch);
+    float* o = out + (size_t)blockIdx.x * hidden;
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x) o[j] = fmaf(gain_b[j], y[j] * fb, gain_a[j] * (x[j] * fa));
+}
+
 inline bool aligned16(const void* p) { return (uintptr_t)p % 16 == 0; }
 inline void warp_rows_launch(int rows, int* blocks, int* threads) {
     const int warps = rows >= 2048 ? 8 : rows >= 512 ? 2 : 1;      // few rows: a warp a block, so that they are spread over the SMs
@@ -478,5 +518,24 @@ EG_API int eg_embedding_gather_scaled(cudaStream_t stream, int dtype, const int*
 EG_API int eg_scale_f32(cudaStream_t stream, float* x, long long n, float s) {
     if (n <= 0) return 0;
     scale_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>(x, n, s);
+    return eg_launch_status();
+}
+
+// out float32 [tokens, hidden] (may be a) = factor * (gain_a a / rms(a) + gain_b b / rms(b)), a and b float32 rows
+EG_API int eg_rmsnorm_pair(cudaStream_t stream, const float* a, const float* b, const float* gain_a, const float* gain_b, float eps, float factor, float* out,
+                           int tokens, int hidden) {
+    if (tokens <= 0) return 0;
+    if (hidden % 4 == 0 && hidden <= 2048 && aligned16(a) && aligned16(b) && aligned16(gain_a) && aligned16(gain_b) && aligned16(out)) {
+        int blocks, threads;
+        warp_rows_launch(tokens, &blocks, &threads);
+        const int vpl = (hidden / 4 + 31) / 32;
+#define EG_PAIR(V) rmsnorm_pair_warp_kernel<V><<<blocks, threads, 0, stream>>>(a, b, gain_a, gain_b, eps, factor, out, tokens, hidden)
+        if (vpl <= 4) EG_PAIR(4);
+        else if (vpl <= 8) EG_PAIR(8);
+        else EG_PAIR(16);
+#undef EG_PAIR
+        return eg_launch_status();
+    }
+    rmsnorm_pair_kernel<<<tokens, row_threads(hidden), 0, stream>>>(a, b, gain_a, gain_b, eps, factor, out, hidden);
     return eg_launch_status();
 }
