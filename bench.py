@@ -31,6 +31,7 @@ For profiling and for further sizes (one short line each, never the JSON line ab
     python bench.py --only gufanex [--batch B] [--context C] [--steps K] [--sizes small|medium]
     python bench.py --only lasizen [--batch B] [--context C] [--steps K] [--sizes small|medium]
     python bench.py --only mozalix [--batch B] [--context C] [--steps K] [--sizes small|medium] [--model both|mozalix|lasizen]
+    python bench.py --only zodosun [--batch B] [--context C] [--steps K] [--sizes small|medium] [--model both|zodosun|mozalix]
 
 `gufanex` measures the Gufanex decoder (selective-scan and latent-attention layers with routed experts) at layer sizes
 of real models of those kinds, with random weights, beside a Qwen2 decoder of the same width, depth and active
@@ -43,6 +44,10 @@ feed-forward weights.
 `mozalix` measures the Mozalix decoder (attention with two softmax maps a head, attention in chunks with sinks, a windowed
 attention that keeps first tokens beside a delta-rule mixer with a decay per key channel, gated feed-forwards with limits and
 biases) the same way, beside the Lasizen decoder of the same width, layer runs and heads.
+
+`zodosun` measures the Zodosun decoder (attention with sigmoid weights and a bias by distance beside a linear attention with a
+fading state, delta-rule mixers with a decay and a removal rate per key channel, norms in groups) the same way, beside the
+Mozalix decoder of the same width, layer runs and feed-forward.
 
 `serve` runs 64 concurrent requests (prompts of 128..4096 tokens in portions of 512 beside
 decoding requests, 512 new tokens each) through the engine and reports wall-clock tokens a second.
@@ -159,6 +164,25 @@ def mozalix_bench_configs(size):
     layers += [dict(layers[j], weights_of=j) for j in range(3)]
     mozalix = {"architecture": "Mozalix", "vocab": 32000, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": float(width) ** 0.5}, "layers": layers}
     return mozalix, lasizen_bench_configs(size)[0]
+
+
+# Layer sizes for `--only zodosun`: width 2,048 in 4 norm groups; delta-rule mixers of 32 heads with 64 x 64 states and decays
+# through maps of inner size 64; a layer of two mixers side by side (an attention with sigmoid weights, 16 heads of 128 over 4 key
+# heads, all earlier keys, a bias by distance up to 1,024, beside a linear attention of 8 heads with 128 x 128 states); SwiGLU
+# feed-forwards of 5,504 ("medium"), and half of the width, heads and feed-forward ("small").  Six layers, two of them with two
+# mixers.  Beside it the closest existing model, the Mozalix decoder of `--only mozalix` (attentions, a side-by-side layer, a
+# delta rule with a decay per key channel): same width, layer runs and feed-forward.
+def zodosun_bench_configs(size):
+    k = {"medium": 1, "small": 2}[size]
+    width = 2048 // k
+    delta = {"type": "general_delta", "mixer": {"heads": 32 // k, "dim": 64, "rank": 64}}
+    pair = {"type": "parallel", "mixer": {"left": {"heads": 16 // k, "kv_heads": 4 // k, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "bias_max": 1024,
+                                                   "q_temp": {"coef": 0.1, "every": 1024}},
+                                          "right": {"heads": 8 // k, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-2 - h) for h in range(8 // k)]}}}
+    mlp = {"kind": "dense", "ff": (8 * width // 3 + 127) // 128 * 128}
+    zodosun = {"architecture": "Zodosun", "vocab": 32000, "width": width, "norm": {"eps": 1e-6, "groups": 4}, "logit_scale": 0.5,
+               "layers": [dict(m, mlp=mlp) for m in (delta, pair, delta, delta, pair, delta)]}
+    return zodosun, mozalix_bench_configs(size)[0]
 
 
 CONTEXT = 4096
@@ -348,6 +372,8 @@ def gufanex_folder(config, seed=0):
         from easy_gpt.cpp_b200.weights.masezen_init import write_random_model
     elif config.get("architecture") == "Mozalix":
         from easy_gpt.cpp_b200.weights.mozalix_init import write_random_model
+    elif config.get("architecture") == "Zodosun":
+        from easy_gpt.cpp_b200.weights.zodosun_init import write_random_model
     else:
         from easy_gpt.cpp_b200.weights.gufanex_init import write_random_model
 
@@ -710,7 +736,25 @@ def run_mozalix(args):
     return 0
 
 
+def run_zodosun(args):
+    size = args.sizes if args.sizes in ("small", "medium") else "medium"
+    zodosun, mozalix = zodosun_bench_configs(size)
+    context = min(args.context, 2048) if args.context == CONTEXT else args.context
+    out = {"only": "zodosun", "sizes": size, "batch": args.batch, "context": context, "prefill_tokens": PREFILL_TOKENS, "dtype": "bfloat16",
+           "data": "synthetic (random weights)"}
+    with ClockSampler() as clocks:
+        if args.model in ("both", "zodosun"):
+            out["zodosun"] = measure_prefill_and_decode(gufanex_folder(zodosun), zodosun["vocab"], args.batch, context, args.steps, args.warmup)
+        if args.model in ("both", "mozalix"):
+            out["mozalix_equal"] = measure_prefill_and_decode(gufanex_folder(mozalix), mozalix["vocab"], args.batch, context, args.steps, args.warmup)
+    out["clocks"] = clocks.summary()
+    print(json.dumps(out))
+    return 0
+
+
 def run_ours(args):
+    if args.only == "zodosun":
+        return run_zodosun(args)
     if args.only == "mozalix":
         return run_mozalix(args)
     if args.only == "gufanex":
@@ -846,16 +890,16 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--context", type=int, default=CONTEXT, help="context length the decode steps end at (default 4096)")
-    ap.add_argument("--sizes", choices=list(SIZES) + ["small", "medium"], default="0.5b", help="layer sizes for --only runs (small, medium: --only gufanex, --only lasizen, --only masezen and --only mozalix)")
-    ap.add_argument("--model", choices=["both", "gufanex", "lasizen", "masezen", "mozalix", "qwen2"], default="both",
-                    help="with --only gufanex, --only lasizen, --only masezen or --only mozalix: which of the two models to measure")
+    ap.add_argument("--sizes", choices=list(SIZES) + ["small", "medium"], default="0.5b", help="layer sizes for --only runs (small, medium: --only gufanex, --only lasizen, --only masezen, --only mozalix and --only zodosun)")
+    ap.add_argument("--model", choices=["both", "gufanex", "lasizen", "masezen", "mozalix", "zodosun", "qwen2"], default="both",
+                    help="with --only gufanex, --only lasizen, --only masezen, --only mozalix or --only zodosun: which of the two models to measure")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16", help="precision of --only decode")
     ap.add_argument("--default-options", action="store_true",
                     help="--only decode with the engine's default page size and request length")
     ap.add_argument("--ref-prompt", type=int, default=0,
                     help="prompt length of the reference arm (0: 1536, or the longest its int-indexed logits allow)")
     ap.add_argument("--fused", action="store_true", help="with --only timeline or decode: the decode step as one persistent kernel (EASY_GPT_FUSED_DECODE=1)")
-    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "gemm", "attention", "serve", "gufanex", "lasizen", "masezen", "mozalix"], default=None,
+    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "gemm", "attention", "serve", "gufanex", "lasizen", "masezen", "mozalix", "zodosun"], default=None,
                     help="measure one part only and print a short line (for profiling runs)")
     args = ap.parse_args()
     if args.gpus != 1:

@@ -41,6 +41,12 @@
 // EG_STATUS_WAIT_TIMEOUT; every role then leaves its loop, the loader waits (bounded again) for the copies it
 // still has in flight, and the TMEM is freed as usual.
 //
+// A third form of the rows (SIGMOID): the weight of a visible key is the sigmoid of its score, the score being scaled and
+// given a bias by distance from a table of the head (entry min(distance, reach - 1), in shared memory), and the rows' sums are
+// multiplied by sigmoid(gate) instead of divided by anything.  No weight depends on another key, so there is no maximum, no
+// reference and no rescaling, and the parts of a cut key range simply add up (they carry reference 0 and sum 1).
+// weight = 1 / (1 + 2^x) with x = -log2(e) s: one exponent a score and one reciprocal for two scores (1 / a = b * 1 / (a b)).
+//
 // Takes head sizes 64 and 128, pages of a multiple of 16 tokens, 16-byte aligned rows.  Anything else:
 // cudaErrorInvalidValue, and the caller uses the warp-level kernel.
 #define EG_NEEDS_TENSOR_MAPS
@@ -239,7 +245,28 @@ struct Params {
     float out_scale = 1.f;
     const float* sinks = nullptr;
     float* out_f32 = nullptr;
+    // SIGMOID: -log2(e) times the bias of every head by distance [num_heads, reach], the gates' logits [tokens, ld_gate] (head h at
+    // column h, or null); `scale` is then -log2(e) times the scores' factor
+    const float* bias_table = nullptr;
+    int reach = 1;
+    const float* gate = nullptr;
+    long long ld_gate = 0;
 };
+enum Form { PLAIN = 0, MASKED_FORM = 1, SIGMOID = 2 };
+constexpr int BIAS_ENTRIES = 2048;                                // of a head's table, in shared memory
+
+// two weights 1 / (1 + 2^x0), 1 / (1 + 2^x1) with one reciprocal (x is kept below 60, where the weight is 1e-18, so that the product
+// of the two denominators stays finite)
+__device__ __forceinline__ void two_weights(float x0, float x1, float& w0, float& w1) {
+    float a, b, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a) : "f"(fminf(x0, 60.f)));
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(b) : "f"(fminf(x1, 60.f)));
+    a += 1.f;
+    b += 1.f;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(a * b));
+    w0 = r * b;
+    w1 = r * a;
+}
 
 // MASKED (a template parameter of the kernels): the further masks are read; without it they are constants ("none"), and the
 // kernels are the plain ones to the instruction.
@@ -267,17 +294,23 @@ __device__ __forceinline__ float norm_with_sink(float m, float l, float sink2) {
     return c / fmaf(l, c, exp2f(sink2 - top));
 }
 
+// SIGMOID: what a head's output is multiplied by
+__device__ __forceinline__ float gate_of(const Params& p, int token, int h, bool valid) {
+    return p.gate && valid ? 1.0f / (1.0f + expf(-p.gate[(size_t)token * p.ld_gate + h])) : 1.0f;
+}
+
 // The 64-bit shared-memory descriptor from its constant high word and a low word (start address, leading offset).
 __device__ __forceinline__ uint64_t desc_from(uint32_t lo, uint32_t hi) {
     uint64_t d;
     asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "r"(lo), "r"(hi));
     return d;
 }
-template <int HD, int WGS, bool MASKED>
+template <int HD, int WGS, int FORM>
 __global__ void __launch_bounds__((Shape<HD, WGS>::THREADS), (Shape<HD, WGS>::CTAS_PER_SM))
 attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                  const __grid_constant__ CUtensorMap map_v, const Params p) {
     using S = Shape<HD, WGS>;
+    constexpr bool MASKED = FORM == MASKED_FORM;
     const int x_keep = MASKED ? p.keep_first : 0, x_maps = MASKED ? p.maps : 1;
     const float x_out_scale = MASKED ? p.out_scale : 1.f;
     float* const x_out_f32 = MASKED ? p.out_f32 : nullptr;
@@ -291,6 +324,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     const uint32_t base = (smem_addr(smem_raw) + 1023u) & ~1023u;
     const uint32_t q_addr = base, ring_addr = base + S::Q_BYTES;
     float* const handover = reinterpret_cast<float*>(smem_raw + (base - smem_addr(smem_raw)) + S::Q_BYTES + STAGES * S::STAGE_BYTES);
+    float* const bias_s = handover + S::HANDOVER_BYTES / 4;       // SIGMOID: the unit's head's table [reach]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
     if (threadIdx.x == 0) {
@@ -508,8 +542,13 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
             const uint32_t o_lane = lane_base + (uint32_t)(S::O_COL + g * HD);
 
             // m: the reference of the exponents, a maximum the row has seen (in scaled base-2 units); l: the sum against it
-            float m = -INFINITY, l = 0.f;
+            float m = FORM == SIGMOID ? 0.f : -INFINITY, l = FORM == SIGMOID ? 1.f : 0.f;
             bool ok = true;
+            if constexpr (FORM == SIGMOID) {                      // the last unit's readers are behind the barrier that ended it
+                const float* table = p.bias_table + (size_t)h * p.reach;
+                for (int i = g * 128 + quad * 32 + lane; i < p.reach; i += WGS * 128) bias_s[i] = __ldg(table + i);
+                asm volatile("bar.sync 2, %0;\n" ::"n"(WGS * 128) : "memory");
+            }
             const bool tracing = p.trace && blockIdx.x == 0 && round == 0 && threadIdx.x == 64;
 #define STAMP(k) if (tracing && i < 32) p.trace[i * 8 + (k)] = clock64();
             for (int i = 0; i < my_tiles; ++i) {
@@ -537,6 +576,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                         }
                     }
                     STAMP(2)
+                    if constexpr (FORM != SIGMOID) {
                     // only a tile that crosses the diagonal, the window's far edge or the end of the portion needs limits
                     // (also a tile with kept first keys, and one in which a chunk of some row of the warp begins)
                     const bool limits = key_base + BN - 1 > warp_lo || quad * 32 + 31 >= count || key_base < first_visible<MASKED>(p, warp_lo + 31) ||
@@ -567,12 +607,13 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                     }
                     // a row that has seen nothing keeps m = -inf: 0 as the reference makes exp(-inf - 0) = 0
                     ref = m == -INFINITY ? 0.f : m;
+                    }
                 }
                 STAMP(3)
                 // Rows whose reference moved scale what they have accumulated so far: the product of the tile before
                 // must be done.  (The barriers take turns like the score buffers: a parity tells two phases apart, not
                 // more, and nobody who waits on one of them is ever further than one phase from it.)
-                if (i > 0 && __any_sync(0xffffffffu, c != 1.f)) {
+                if (FORM != SIGMOID && i > 0 && __any_sync(0xffffffffu, c != 1.f)) {
                     ok = __all_sync(0xffffffffu, mbar_wait(&o_done[g * SCORE_BUFFERS + (n - 1) % SCORE_BUFFERS], ((n - 1) / SCORE_BUFFERS) & 1, &abort_flag, p.status));
                     if (!ok) break;
                     tc_fence_after();
@@ -603,6 +644,27 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                     if (skip) {
 #pragma unroll
                         for (int e = 0; e < 16; ++e) packed[e] = 0u;
+                    } else if constexpr (FORM == SIGMOID) {
+                        // distance of element k: near - k.  A tile whose keys all lie at least `last` back has one bias a row.
+                        const int near = qpos - key_base - 32 * half, last = p.reach - 1;
+                        if (warp_lo - (key_base + BN - 1) >= last && quad * 32 + 31 < count) {
+                            const float b = bias_s[last];
+#pragma unroll
+                            for (int e = 0; e < 16; ++e) {
+                                float w0, w1;
+                                two_weights(fmaf(s[32 * half + 2 * e], p.scale, b), fmaf(s[32 * half + 2 * e + 1], p.scale, b), w0, w1);
+                                packed[e] = pack2(w0, w1);
+                            }
+                        } else {
+#pragma unroll
+                            for (int e = 0; e < 16; ++e) {
+                                const int n0 = near - 2 * e, n1 = n0 - 1;
+                                float w0, w1;
+                                two_weights(fmaf(s[32 * half + 2 * e], p.scale, bias_s[max(min(n0, last), 0)]),
+                                            fmaf(s[32 * half + 2 * e + 1], p.scale, bias_s[max(min(n1, last), 0)]), w0, w1);
+                                packed[e] = pack2(valid && n0 >= 0 ? w0 : 0.f, valid && n1 >= 0 ? w1 : 0.f);
+                            }
+                        }
                     } else {
 #pragma unroll
                         for (int e = 0; e < 16; ++e) {
@@ -617,7 +679,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 }
                 float sum0, sum1;
                 split_pair(sums, sum0, sum1);
-                l = l * c + (sum0 + sum1);
+                if (FORM != SIGMOID) l = l * c + (sum0 + sum1);
                 STAMP(5)
                 tmem_st_wait();
                 STAMP(6)
@@ -683,7 +745,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 // the second group's rows are with the first
             } else if (ok && parts == 1) {
                 tc_fence_after();
-                const float inv = norm_with_sink(m, l, sink_of<MASKED>(p, h)) * x_out_scale;
+                const float inv = FORM == SIGMOID ? gate_of(p, t0 + row, h, valid) : norm_with_sink(m, l, sink_of<MASKED>(p, h)) * x_out_scale;
                 const size_t at = (size_t)(t0 + row) * p.ldo + (size_t)h * HD;
                 uint4* dst = reinterpret_cast<uint4*>(p.out + at);
                 float4* dst32 = reinterpret_cast<float4*>(x_out_f32 + at);
@@ -756,9 +818,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
 // Adds up the parts of the query tiles whose key ranges were cut: one CTA per (query tile, head), a thread per
 // (row, 16 columns); every part's numbers are requested before the first is used.
 constexpr int MERGE_MAX_PARTS = 8;
-template <int HD, bool MASKED>
+template <int HD, int FORM>
 __global__ void __launch_bounds__(256)
 attention_merge_parts_kernel(const Params p) {
+    constexpr bool MASKED = FORM == MASKED_FORM;
     const float x_out_scale = MASKED ? p.out_scale : 1.f;
     float* const x_out_f32 = MASKED ? p.out_f32 : nullptr;
     asm volatile("griddepcontrol.wait;\n" ::: "memory");
@@ -794,7 +857,7 @@ attention_merge_parts_kernel(const Params p) {
             w[i] = ml[i].x == -INFINITY ? 0.f : exp2f(ml[i].x - big);                     // -inf: that part saw no key of this row
             total += w[i] * ml[i].y;
         }
-        const float inv = norm_with_sink(big, total, sink_of<MASKED>(p, h)) * x_out_scale;
+        const float inv = FORM == SIGMOID ? gate_of(p, t0 + row, h, true) : norm_with_sink(big, total, sink_of<MASKED>(p, h)) * x_out_scale;
         float acc[16];
 #pragma unroll
         for (int e = 0; e < 16; ++e) acc[e] = 0.f;
@@ -834,18 +897,19 @@ int make_map(CUtensorMap* map, const void* base, long long rows, long long cols,
     return r == CUDA_SUCCESS ? 0 : (int)cudaErrorInvalidValue;
 }
 
-template <int HD, int WGS, bool MASKED>
+template <int HD, int WGS, int FORM>
 int launch(cudaStream_t stream, const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v, const Params& p, int sm_count) {
     using S = Shape<HD, WGS>;
+    constexpr int smem = S::SMEM_BYTES + (FORM == SIGMOID ? BIAS_ENTRIES * 4 : 0);
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tcgen05_kernel<HD, WGS, MASKED>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::SMEM_BYTES);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tcgen05_kernel<HD, WGS, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     const long long units = (long long)p.num_tiles * p.num_heads * p.max_parts, places = (long long)S::CTAS_PER_SM * sm_count;
     const int ctas = (int)(units < places ? units : places);
-    attention_prefill_tcgen05_kernel<HD, WGS, MASKED><<<ctas, S::THREADS, S::SMEM_BYTES, stream>>>(map_q, map_k, map_v, p);
+    attention_prefill_tcgen05_kernel<HD, WGS, FORM><<<ctas, S::THREADS, smem, stream>>>(map_q, map_k, map_v, p);
     return eg_launch_status();
 }
 
@@ -908,6 +972,10 @@ static int attention_prefill_tcgen05_any(cudaStream_t stream, const void* q, lon
         p.out_scale = extras->out_scale;
         p.sinks = extras->sinks;
         p.out_f32 = extras->out_f32;
+        p.bias_table = extras->bias_table;
+        p.reach = extras->reach;
+        p.gate = extras->gate;
+        p.ld_gate = extras->ld_gate;
     }
     // rows of head_dim elements that the cache maps cover: up to the last row of the last page
     const long long kv_rows = (long long)(num_pages - 1) * p.page_rows + (long long)(num_kv_heads - 1) * p.head_rows + page_size;
@@ -929,11 +997,11 @@ static int attention_prefill_tcgen05_any(cudaStream_t stream, const void* q, lon
     static const int asked = getenv("EASY_GPT_PREFILL_GROUPS") ? atoi(getenv("EASY_GPT_PREFILL_GROUPS")) : 0;
     const int groups = asked == 1 || asked == 2 ? asked : eg_attention_prefill_groups(head_dim);
     int code;
-    const bool masked = extras != nullptr;
-    if (groups == 1 && masked) code = head_dim == 64 ? launch<64, 1, true>(stream, map_q, map_k, map_v, p, sm_count) : launch<128, 1, true>(stream, map_q, map_k, map_v, p, sm_count);
-    else if (groups == 1) code = head_dim == 64 ? launch<64, 1, false>(stream, map_q, map_k, map_v, p, sm_count) : launch<128, 1, false>(stream, map_q, map_k, map_v, p, sm_count);
-    else if (masked) code = head_dim == 64 ? launch<64, 2, true>(stream, map_q, map_k, map_v, p, sm_count) : launch<128, 2, true>(stream, map_q, map_k, map_v, p, sm_count);
-    else code = head_dim == 64 ? launch<64, 2, false>(stream, map_q, map_k, map_v, p, sm_count) : launch<128, 2, false>(stream, map_q, map_k, map_v, p, sm_count);
+    const int form = !extras ? PLAIN : extras->bias_table ? SIGMOID : MASKED_FORM;
+#define EG_FORM(WGS, F) (head_dim == 64 ? launch<64, WGS, F>(stream, map_q, map_k, map_v, p, sm_count) : launch<128, WGS, F>(stream, map_q, map_k, map_v, p, sm_count))
+    if (groups == 1) code = form == SIGMOID ? EG_FORM(1, SIGMOID) : form == MASKED_FORM ? EG_FORM(1, MASKED_FORM) : EG_FORM(1, PLAIN);
+    else code = form == SIGMOID ? EG_FORM(2, SIGMOID) : form == MASKED_FORM ? EG_FORM(2, MASKED_FORM) : EG_FORM(2, PLAIN);
+#undef EG_FORM
     if (code || max_parts == 1) return code;
     // the parts are added up behind the main kernel (launched early: it waits for it by itself)
     cudaLaunchConfig_t cfg = {};
@@ -945,11 +1013,13 @@ static int attention_prefill_tcgen05_any(cudaStream_t stream, const void* q, lon
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    if (masked)
-        return (int)(head_dim == 64 ? cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<64, true>, p)
-                                    : cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<128, true>, p));
-    return (int)(head_dim == 64 ? cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<64, false>, p)
-                                : cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<128, false>, p));
+#define EG_MERGE(F)                                                                              \
+    return (int)(head_dim == 64 ? cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<64, F>, p) \
+                                : cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<128, F>, p))
+    if (form == SIGMOID) EG_MERGE(SIGMOID);
+    if (form == MASKED_FORM) EG_MERGE(MASKED_FORM);
+    EG_MERGE(PLAIN);
+#undef EG_MERGE
 }
 
 EG_API int eg_attention_prefill_tcgen05(cudaStream_t stream, const void* q, long long ldq, int total_tokens, const void* k_cache,
@@ -995,4 +1065,25 @@ EG_API int eg_attention_prefill_tcgen05_masked(cudaStream_t stream, const void* 
     return attention_prefill_tcgen05_any(stream, q, ldq, total_tokens, k_cache, v_cache, block_table, table_stride, positions, tiles, num_tiles, out, ldo,
                                          num_heads, num_kv_heads, head_dim, page_size, page_stride, head_stride, num_pages, window, scale, status, nullptr,
                                          max_parts, part_tiles, partial_o, partial_ml, queue, -INFINITY, &extras);
+}
+
+// How many entries of a head's bias table the sigmoid form keeps in shared memory (a longer reach: the caller uses another kernel).
+EG_API int eg_attention_prefill_tcgen05_sigmoid_reach(void) { return BIAS_ENTRIES; }
+
+// The sigmoid form: weights sigmoid(score * scale + bias(distance)), not normalised.  bias_table float32 [num_heads, reach] times -log2(e)
+// (natural units times that), reach up to the above; gate float32 [tokens, ld_gate] (head h at column h) or null; bfloat16 output.
+EG_API int eg_attention_prefill_tcgen05_sigmoid(cudaStream_t stream, const void* q, long long ldq, int total_tokens, const void* k_cache, const void* v_cache,
+                                                const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, void* out,
+                                                long long ldo, int num_heads, int num_kv_heads, int head_dim, int page_size, long long page_stride,
+                                                long long head_stride, int num_pages, float scale, const float* bias_table, int reach, const float* gate,
+                                                long long ld_gate, int* status, int max_parts, int part_tiles, float* partial_o, float* partial_ml, int* queue) {
+    if (!bias_table || reach < 1 || reach > BIAS_ENTRIES) return (int)cudaErrorInvalidValue;
+    Params extras{};
+    extras.bias_table = bias_table;
+    extras.reach = reach;
+    extras.gate = gate;
+    extras.ld_gate = ld_gate;
+    return attention_prefill_tcgen05_any(stream, q, ldq, total_tokens, k_cache, v_cache, block_table, table_stride, positions, tiles, num_tiles, out, ldo,
+                                         num_heads, num_kv_heads, head_dim, page_size, page_stride, head_stride, num_pages, 0, -1.4426950408889634f * scale, status,
+                                         nullptr, max_parts, part_tiles, partial_o, partial_ml, queue, -INFINITY, &extras);
 }

@@ -23,6 +23,8 @@ struct SubLayer {
     std::shared_ptr<Mixer> mixer;
     std::shared_ptr<FeedForward> feed_forward;
     bool plain_pre_norm = false;        // x = x + part(norm(x)) with nothing behind the part: the shape whose add and norm the parts may fuse
+    // whether the sub-layer in front may prepare this one's norm: the part must take a norm that is not computed yet
+    bool takes_prepared_norm() const { return plain_pre_norm && (mixer ? mixer->accepts_pending_norm() : feed_forward->accepts_pending_norm()); }
     Part* part() const { return mixer ? static_cast<Part*>(mixer.get()) : static_cast<Part*>(feed_forward.get()); }
     std::vector<Part*> parts() const {
         std::vector<Part*> out;
@@ -77,7 +79,7 @@ public:
         return n;
     }
     // the norm that a fused add + norm in front of this layer would have to be (nullptr: nothing in front may prepare it)
-    const Norm* first_norm() const { return !parallel && sublayers.front().plain_pre_norm ? sublayers.front().norm.get() : nullptr; }
+    const Norm* first_norm() const { return !parallel && sublayers.front().takes_prepared_norm() ? sublayers.front().norm.get() : nullptr; }
 
     // The residual stream between layers: the buffer that holds it, a second buffer of its size, and what is still to be
     // added to it (a part's output, or two of them behind a parallel layer; the norm that comes next adds them).
@@ -233,7 +235,7 @@ public:
             // this sub-layer's arena: what the sub-layer before the last one left there is dead by now
             ctx.arena = &arenas.sub[(*turn)++ & 1];
             ctx.arena->reset();
-            const Norm* following = (i + 1 < sublayers.size()) ? (sublayers[i + 1].plain_pre_norm ? sublayers[i + 1].norm.get() : nullptr) : next_norm;
+            const Norm* following = (i + 1 < sublayers.size()) ? (sublayers[i + 1].takes_prepared_norm() ? sublayers[i + 1].norm.get() : nullptr) : next_norm;
             const int hidden = sub.norm ? sub.norm->size() : width_;
             if (sub.plain_pre_norm) {
                 const int fused_rows = plans::fused_norm_max_tokens(sub.norm->size());

@@ -60,7 +60,8 @@ private:
 // weight = sigmoid(score), not normalised;  out = W_o (heads' sums times sigmoid(gate_h), side by side).
 // Without `distance_bias` there is no .rel, without `head_bias` no .pb, without `head_gate` no .g, without `proj_bias` no biases.
 // The cache keeps one row (key | value) per token and key head, where dim = vdim planes of their own.  float32 and sizes that are
-// no multiples of 8 run on the generic kernel; bfloat16 runs on the tensor cores (attention_sigmoid.cu).
+// no multiples of 8 run on the generic kernel; bfloat16 runs on the tensor cores (attention_tcgen05.cu for longer prompt portions of
+// heads of 64 and 128, else attention_sigmoid.cu).
 // Parameters: hidden_size, heads, kv_heads, dim, vdim, scale, norm_eps, temp_coef, temp_every, bias_max, distance_bias, head_bias,
 // head_gate, proj_bias.  Tensors: .q .k .v .o (+ .q.b .k.b .v.b, .q.norm .k.norm, .rel, .pb, .g).
 class SigmoidAttention : public Mixer {
@@ -175,11 +176,30 @@ public:
         Rows attn{ctx.take_rows(T, heads_ * dv_, dtype), dtype, T, heads_ * dv_, heads_ * dv_};
         const float* gate = head_gate_ ? (const float*)proj.p + (size_t)(heads_ + kv_heads_) * dk_ + (size_t)kv_heads_ * dv_ : nullptr;
         if (mma_ && cache.head_stride % 8 == 0 && cache.page_stride % 8 == 0) {
-            if (ctx.query_tiles)
+            // prompt portions in tiles of query tokens: on tcgen05 where they are long enough to fill its 128-row tiles (heads of 64 and 128,
+            // keys and values of one size), else on the warp-level tensor cores; single tokens split over their keys
+            if (ctx.query_tiles && planes() && reach_ <= eg_attention_prefill_tcgen05_sigmoid_reach() && ctx.max_query_len >= plans::TCGEN05_ATTENTION_MIN_QUERY &&
+                plans::attention_prefill_tcgen05_takes(dtype, dk_, cache.page_size)) {
+                int parts, part_tiles;
+                plans::attention_prefill_parts(ctx.num_tiles, heads_, dk_, ctx.max_context_len, &parts, &part_tiles);
+                const size_t slots = (size_t)ctx.num_tiles * heads_;
+                while (parts > 1 && slots * parts * 128 * (dk_ + 2) * 4 > plans::PREFILL_PARTS_SCRATCH_BYTES) --parts;
+                float *partial_o = nullptr, *partial_ml = nullptr;
+                if (parts > 1) {
+                    partial_o = ctx.take<float>(slots * parts * 128 * dk_);
+                    partial_ml = ctx.take<float>(slots * parts * 128 * 2);
+                }
+                launch_check(eg_attention_prefill_tcgen05_sigmoid(ctx.stream, q.p, q.ld, T, cache.k, cache.v, tables.block_table, tables.table_width, ctx.positions,
+                                                                  ctx.query_tiles, ctx.num_tiles, attn.p, attn.ld, heads_, kv_heads_, dk_, cache.page_size,
+                                                                  cache.page_stride, cache.head_stride, cache.num_pages, scale_, table_.as<float>(), reach_, gate,
+                                                                  proj.ld, ctx.status, parts, part_tiles, partial_o, partial_ml,
+                                                                  ctx.scratch->prefill_queue.as<int>()), "attention_prefill_tcgen05_sigmoid");
+            } else if (ctx.query_tiles) {
                 launch_check(eg_sigmoid_attention_tiles(ctx.stream, q.p, cache.k, values, row_stride, cache.head_stride, tables.block_table, tables.table_width,
                                                         ctx.positions, ctx.query_tiles, ctx.num_tiles, table_.as<float>(), reach_, gate, proj.ld, attn.p, attn.ld,
                                                         heads_, kv_heads_, dk_, dv_, cache.page_size, cache.page_stride, cache.num_pages, scale_, ctx.status),
                              "sigmoid_attention_tiles");
+            }
             const int singles = ctx.query_tiles ? ctx.num_small : T;
             if (singles > 0) {
                 const int blocks = (heads_ / kv_heads_ + 15) / 16 * kv_heads_;
@@ -233,7 +253,7 @@ public:
           dv_((int)p.integer("vdim")), eps_((float)p.real("eps")) {
         if (hidden_ <= 0 || heads_ <= 0 || dk_ <= 0 || dv_ <= 0) throw std::invalid_argument("lightning attention: sizes must be positive");
         if (dk_ > 256) throw std::invalid_argument("lightning attention: dim up to 256 is what the kernel takes");
-        for (int h = 0; h < heads_; ++h) decays_.push_back((float)p.real("decay." + std::to_string(h)));
+        for (int h = 0; h < heads_; ++h) decays_.push_back(p.real("decay." + std::to_string(h)));
     }
     std::vector<TensorRequest> tensor_requests() const override {
         const long long k = (long long)heads_ * dk_, v = (long long)heads_ * dv_;
@@ -246,11 +266,17 @@ public:
         in_ = Linear(w.data(), rows, hidden_, nullptr, dtype);
         out_ = Linear(need_tensor(file, prefix + ".o"), nullptr, dtype);
         norm_w_ = upload_f32(file, prefix + ".norm");
-        decay_ = upload(decays_.data(), decays_.size(), DType::F32);
+        std::vector<float> powers;                                            // of every head's decay, from 0 to 64
+        for (double d : decays_) {
+            double x = 1.0;
+            for (int i = 0; i <= 64; ++i, x *= d) powers.push_back((float)x);
+        }
+        powers_ = upload(powers.data(), powers.size(), DType::F32);
     }
     size_t weight_bytes() const override { return in_.weight_bytes() + out_.weight_bytes(); }
     size_t arena_bytes(long long T) const override {
-        return (size_t)T * ((size_t)in_.out_features * 4 + (size_t)heads_ * dv_ * 8 + (size_t)hidden_ * 4) + (1u << 16);
+        const size_t chunks = (size_t)(T / 64 + T / 32 + 1) * heads_ * dv_ * dk_ * 4;
+        return (size_t)T * ((size_t)in_.out_features * 4 + (size_t)heads_ * dv_ * 8 + (size_t)hidden_ * 4) + chunks + (1u << 16);
     }
     bool capturable() const override { return true; }
     long long slot_floats() const { return (long long)heads_ * dv_ * dk_; }
@@ -266,8 +292,10 @@ public:
         Rows y{ctx.take_rows(T, heads_ * dv_, dtype), dtype, T, heads_ * dv_, heads_ * dv_};
         float* o_raw = ctx.take<float>((size_t)T * heads_ * dv_);
         const int k = heads_ * dk_, v = heads_ * dv_;
-        launch_check(eg_lightning(ctx.stream, (const float*)proj.p, proj.ld, 0, k, 2 * k, 2 * k + v, decay_.as<float>(), norm_w_.as<float>(), (float*)cache.state,
-                                  slot_floats(), 0, ctx.seq_starts, ctx.seq_slots, o_raw, y.p, (int)dtype, y.ld,
+        const long long in_chunks = eg_lightning_chunk_floats(T, ctx.num_seqs, ctx.max_query_len, heads_, dk_, dv_);
+        float* chunks = in_chunks > 0 ? ctx.take<float>((size_t)in_chunks) : nullptr;
+        launch_check(eg_lightning(ctx.stream, (const float*)proj.p, proj.ld, 0, k, 2 * k, 2 * k + v, powers_.as<float>(), norm_w_.as<float>(), (float*)cache.state,
+                                  slot_floats(), 0, ctx.seq_starts, ctx.seq_slots, o_raw, chunks, y.p, (int)dtype, y.ld,
                                   plans::delta_column_slices(ctx.num_seqs, heads_, dv_), T, ctx.num_seqs, heads_, dk_, dv_, eps_), "lightning");
         const Rows o = out_(ctx, y, /*out_f32=*/true);
         Delta d;
@@ -279,9 +307,9 @@ public:
 private:
     int hidden_, heads_, dk_, dv_;
     float eps_;
-    std::vector<float> decays_;
+    std::vector<double> decays_;
     Linear in_, out_;
-    DeviceBuffer norm_w_, decay_;
+    DeviceBuffer norm_w_, powers_;
 };
 
 // ---- the generalised delta rule ---------------------------------------------------------------------------------------------------
@@ -328,7 +356,7 @@ public:
     }
     size_t weight_bytes() const override { return in_.weight_bytes() + w2_.weight_bytes() + out_.weight_bytes(); }
     size_t arena_bytes(long long T) const override {
-        return (size_t)T * ((size_t)in_.out_features * 4 + (size_t)padded(rank_) * 4 + (size_t)heads_ * dim_ * (4 + 12 + 4 + 4) + (size_t)hidden_ * 4) + (1u << 16);
+        return (size_t)T * ((size_t)in_.out_features * 4 + (size_t)padded(rank_) * 4 + (size_t)heads_ * (dim_ * (4 + 4 + 4) + eg_general_delta_record(dim_) * 4) + (size_t)hidden_ * 4) + (1u << 16);
     }
     bool capturable() const override { return true; }
     long long slot_floats() const { return (long long)heads_ * dim_ * dim_; }
@@ -341,16 +369,21 @@ public:
         if (!cache.writes) throw DeviceError("a general delta mixer cannot read another entry's state without advancing it");
         const Rows h = in.pending ? in.pending->materialize() : in.rows;
         const Rows proj = in_(ctx, h, /*out_f32=*/true);                      // [T, r | k | v | g | a' | w'] float32
-        Rows inner{ctx.take_rows(T, w2_.in_features, dtype), dtype, T, w2_.in_features, w2_.in_features};
-        launch_check(eg_tanh_columns(ctx.stream, (const float*)proj.p + 5 * (size_t)n, proj.ld, inner.p, (int)dtype, inner.ld, T, rank_, w2_.in_features), "tanh_columns");
-        const Rows x = w2_(ctx, inner, /*out_f32=*/true);                     // the decays' logits
+        // the decays' logits: a product of its own, or, in steps whose entries are a few tokens each, worked out by the recurrence's blocks
+        Rows x;
+        float* records = nullptr;
+        if (!eg_general_delta_inline_takes(ctx.max_query_len, rank_)) {
+            Rows inner{ctx.take_rows(T, w2_.in_features, dtype), dtype, T, w2_.in_features, w2_.in_features};
+            launch_check(eg_tanh_columns(ctx.stream, (const float*)proj.p + 5 * (size_t)n, proj.ld, inner.p, (int)dtype, inner.ld, T, rank_, w2_.in_features), "tanh_columns");
+            x = w2_(ctx, inner, /*out_f32=*/true);
+            records = ctx.take<float>((size_t)T * heads_ * eg_general_delta_record(dim_));
+        }
         Rows y{ctx.take_rows(T, n, dtype), dtype, T, n, n};
-        float* vecs = ctx.take<float>((size_t)T * n * 3);
         float* o_raw = ctx.take<float>((size_t)T * n);
-        launch_check(eg_general_delta(ctx.stream, (const float*)proj.p, proj.ld, 0, n, 2 * n, 3 * n, 4 * n, (const float*)x.p, x.ld, w0_.as<float>(), a0_.as<float>(),
-                                      norm_w_.as<float>(), vecs, (float*)cache.state, slot_floats(), 0, ctx.seq_starts, ctx.seq_slots, y.p, (int)dtype, y.ld, o_raw,
-                                      plans::delta_column_slices(ctx.num_seqs, heads_, dim_), T, ctx.num_seqs, heads_, dim_, unit_eps_, eps_, decay_scale_),
-                     "general_delta");
+        launch_check(eg_general_delta(ctx.stream, (const float*)proj.p, proj.ld, 0, n, 2 * n, 3 * n, 4 * n, 5 * n, (const float*)x.p, x.ld, w2_.weight,
+                                      w2_.in_features, rank_, w0_.as<float>(), a0_.as<float>(), norm_w_.as<float>(), records, (float*)cache.state, slot_floats(), 0,
+                                      ctx.seq_starts, ctx.seq_slots, y.p, (int)dtype, y.ld, o_raw, plans::general_delta_slices(ctx.num_seqs, heads_, dim_), T,
+                                      ctx.num_seqs, heads_, dim_, unit_eps_, eps_, decay_scale_, ctx.status), "general_delta");
         const Rows o = out_(ctx, y, /*out_f32=*/true);
         Delta d;
         d.p = o.p;

@@ -7,76 +7,146 @@
 //   S <- diag(w) S - (a u)(u^T S) + k v^T;   o = S^T r                                    (o reads the new state)
 //   out = o / sqrt(mean(o^2) + eps) * gain * sigmoid(g)                                  (mean per head, gain per head and channel)
 //
-// r, k, v, y and g are columns of one projection's float32 output, x comes from a second product.
+// r, k, v, y and g are columns of one projection's float32 output; x = W_2 tanh(the projection's last columns).
 //
-// A kernel over all tokens first makes w, u and a u (a warp per token and head).  Then one block per (head, batch entry,
-// slice of the head's columns: the columns of S do not depend on one another).  COLS neighbouring columns of S belong to P
-// neighbouring lanes, each with R of their rows in registers for the entry's whole run of tokens.  Per token a lane reads its
-// rows' pieces of five vectors (w, u, a u, k, r) from shared memory once for all its columns; the dot product with u over the
-// old rows is the only thing the next step waits for, the one with r over the new rows is not.  The block walks the entry in
-// tiles of tokens that arrive by asynchronous copies, the next tile's behind this one's steps.  Outputs are normed and gated by the
-// block itself where it holds a whole head, else by a kernel behind.  The slot keeps S as [head, column, row].  The order of
-// every sum depends on the sizes alone.
+// The recurrence reads a *record* per token and head: the six vectors w, u, a u, k, r, v, each filled up with zeros to DS = R * P
+// values.  Records of a head lie one behind the other, so that a tile of tokens is ONE bulk copy; a kernel over all tokens makes
+// them (a group of lanes per token and head).  In steps whose entries are a few tokens each (decoding) the recurrence's own blocks make
+// them in shared memory, and work out x as well (W_2 is small), which saves two kernels and a product.
+//
+// Recurrence: one block per (head, batch entry, slice of the head's columns: the columns of S do not depend on one another).  A
+// column of S belongs to P neighbouring lanes, each with R of its rows in registers for the entry's whole run of tokens (lane p
+// has rows 4 (i P + p) .. + 3: neighbouring lanes read neighbouring 16-byte pieces).  Per token the dot product with u over the old
+// rows is the only thing the next token waits for: R/4 dependent multiply-adds and log2 P shuffles; decay, value and the dot
+// product with r run beside them, all on pairs of float32.  Tiles arrive three stages ahead.  Outputs are normed and gated by the
+// block where it holds a whole head, else by a kernel behind.  The slot keeps S as [head, column, row].  The order of every sum
+// depends on the sizes alone.
 #include <algorithm>
 #include <cstdlib>
 
 #include "common.cuh"
 #include "decay_exp.cuh"
+#include "mbarrier.cuh"
 
 namespace {
 
-constexpr int PAD = 4;          // floats between the parts' pieces of a staged vector: the parts' 16-byte loads then hit different banks
-constexpr int VECS = 5;         // staged vectors a token: w, u, a u, k, r
+constexpr int VECS = 6, STAGES = 3;
+constexpr unsigned WAIT_LIMIT = 1u << 24;
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ void copy_async_16(float* dst, const float* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
 }
-__device__ __forceinline__ void copy_async_4(float* dst, const float* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ uint64_t pair_of(float lo, float hi) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float sum_of(uint64_t v) {
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+    return lo + hi;
+}
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n"
+                 ::"r"(smem_addr(dst)), "l"(src), "r"(bytes), "r"(smem_addr(bar)) : "memory");
 }
 
 struct DeltaParams {
     const float* proj;          // [tokens, ldp]
     long long ldp;
-    int r_col, k_col, v_col, g_col, a_col;
-    const float* x;             // decays' logits [tokens, ldx], heads x dim
+    int r_col, k_col, v_col, g_col, a_col, inner_col;
+    const float* x;             // decays' logits [tokens, ldx], heads x dim; null: worked out from w2 by the recurrence's blocks
     long long ldx;
+    const void* w2;             // [heads * dim, ld2] in w2's dtype
+    int ld2, rank;
     const float *w0, *a0, *gain;
-    float* vecs;                // [tokens, heads, 3, dim]: w, u, a u
+    float* records;             // [heads, tokens, VECS, DS]
     float* state;
     long long slot_floats, state_offset;
     const int *seq_starts, *seq_slots;
     void* y;
     long long ldy;
     float* o_raw;               // [tokens, heads * dim], or null: the block holds whole heads
-    int tokens, heads, dim, cols, tile, wide;
+    int tokens, heads, dim, cols, tile, lanes;      // lanes: of the group that makes a record
     float unit_eps, eps, decay_scale;
+    int* status;
 };
 
-// a warp per (token, head)
-__global__ void __launch_bounds__(128) general_delta_prepare_kernel(const DeltaParams p) {
-    const int lane = threadIdx.x & 31;
-    const long long i = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (i >= (long long)p.tokens * p.heads) return;
-    const int t = (int)(i / p.heads), h = (int)(i % p.heads), at = h * p.dim;
+// one channel's six values, into rec[v * DS + d]
+__device__ __forceinline__ void put_channel(const DeltaParams& p, const float* row, int at, int d, float x, float inv, float* rec, int DS) {
+    const float k = row[p.k_col + at + d], u = k * inv;
+    rec[d] = decay_exp(-p.decay_scale * sigmoid_f(x + p.w0[at + d]));
+    rec[DS + d] = u;
+    rec[2 * DS + d] = sigmoid_f(row[p.a_col + at + d] + p.a0[at + d]) * u;
+    rec[3 * DS + d] = k;
+    rec[4 * DS + d] = row[p.r_col + at + d];
+    rec[5 * DS + d] = row[p.v_col + at + d];
+}
+
+// `lanes` (a power of two up to 32) neighbouring lanes make the record of a (head, token).  WIDE: four channels a lane and pass, by
+// 16-byte loads and stores.
+template <bool WIDE>
+__global__ void __launch_bounds__(256) general_delta_records_kernel(const DeltaParams p, int DS) {
+    const int group = p.lanes, lane = threadIdx.x % group;
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / group;
+    const bool live = i < (long long)p.tokens * p.heads;
+    // neighbouring groups take neighbouring heads of a token: the projection's rows are read in order
+    const int t = live ? (int)(i / p.heads) : 0, h = live ? (int)(i % p.heads) : 0, at = h * p.dim;
     const float* row = p.proj + (size_t)t * p.ldp;
+    float* rec = p.records + ((size_t)h * p.tokens + t) * VECS * DS;
     float kk = 0.f;
-    for (int d = lane; d < p.dim; d += 32) {
-        const float k = row[p.k_col + at + d];
-        kk = fmaf(k, k, kk);
+    if (WIDE) {
+        for (int d = lane * 4; d < p.dim; d += group * 4) {
+            const float4 k = *reinterpret_cast<const float4*>(row + p.k_col + at + d);
+            kk += k.x * k.x + k.y * k.y + k.z * k.z + k.w * k.w;
+        }
+    } else {
+        for (int d = lane; d < p.dim; d += group) {
+            const float k = row[p.k_col + at + d];
+            kk = fmaf(k, k, kk);
+        }
     }
-    const float inv = 1.0f / sqrtf(warp_sum(kk) + p.unit_eps);
-    float* out = p.vecs + (size_t)i * 3 * p.dim;
-    for (int d = lane; d < p.dim; d += 32) {
-        const float u = row[p.k_col + at + d] * inv;
-        out[d] = decay_exp(-p.decay_scale * sigmoid_f(p.x[(size_t)t * p.ldx + at + d] + p.w0[at + d]));
-        out[p.dim + d] = u;
-        out[2 * p.dim + d] = sigmoid_f(row[p.a_col + at + d] + p.a0[at + d]) * u;
+    for (int o = group >> 1; o > 0; o >>= 1) kk += __shfl_xor_sync(0xffffffffu, kk, o);
+    if (!live) return;
+    const float inv = 1.0f / sqrtf(kk + p.unit_eps);
+    if (WIDE) {
+        for (int d = lane * 4; d < DS; d += group * 4) {
+            float4 v[VECS];
+            if (d < p.dim) {
+                auto load = [&](const float* src) { return *reinterpret_cast<const float4*>(src + at + d); };
+                const float4 x = load(p.x + (size_t)t * p.ldx), w0 = load(p.w0), a = load(row + p.a_col), a0 = load(p.a0);
+                v[3] = load(row + p.k_col);
+                v[4] = load(row + p.r_col);
+                v[5] = load(row + p.v_col);
+                auto decay = [&](float l) { return decay_exp(-p.decay_scale * sigmoid_f(l)); };
+                v[0] = make_float4(decay(x.x + w0.x), decay(x.y + w0.y), decay(x.z + w0.z), decay(x.w + w0.w));
+                v[1] = make_float4(v[3].x * inv, v[3].y * inv, v[3].z * inv, v[3].w * inv);
+                v[2] = make_float4(sigmoid_f(a.x + a0.x) * v[1].x, sigmoid_f(a.y + a0.y) * v[1].y, sigmoid_f(a.z + a0.z) * v[1].z, sigmoid_f(a.w + a0.w) * v[1].w);
+            } else {
+#pragma unroll
+                for (int q = 0; q < VECS; ++q) v[q] = make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int q = 0; q < VECS; ++q) *reinterpret_cast<float4*>(rec + q * DS + d) = v[q];
+        }
+    } else {
+        for (int d = lane; d < DS; d += group) {
+            if (d < p.dim) put_channel(p, row, at, d, p.x[(size_t)t * p.ldx + at + d], inv, rec, DS);
+            else
+                for (int q = 0; q < VECS; ++q) rec[q * DS + d] = 0.f;
+        }
     }
 }
 
-// y = o / rms(o) * gain * sigmoid(g), o dim values in shared or global memory, a warp
+// y = o / rms(o) * gain * sigmoid(g), a warp per (token, head)
 template <typename TO>
 __device__ __forceinline__ void norm_and_gate(const DeltaParams& p, const float* o, size_t t, int h, int lane) {
     float ss = 0.f;
@@ -87,179 +157,241 @@ __device__ __forceinline__ void norm_and_gate(const DeltaParams& p, const float*
     for (int d = lane; d < p.dim; d += 32) out[d] = from_f32<TO>(o[d] * inv * p.gain[h * p.dim + d] * sigmoid_f(g[d]));
 }
 
-template <typename TO>
-__global__ void __launch_bounds__(128) general_delta_output_kernel(const DeltaParams p) {
-    const long long i = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (i >= (long long)p.tokens * p.heads) return;
-    norm_and_gate<TO>(p, p.o_raw + (size_t)i * p.dim, (size_t)(i / p.heads), (int)(i % p.heads), threadIdx.x & 31);
+// behind a recurrence whose blocks held slices of a head: `lanes` lanes per (token, head), four channels a lane and pass (WIDE)
+template <typename TO, bool WIDE>
+__global__ void __launch_bounds__(256) general_delta_output_kernel(const DeltaParams p) {
+    if (!WIDE) {
+        const long long i = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+        if (i >= (long long)p.tokens * p.heads) return;
+        norm_and_gate<TO>(p, p.o_raw + (size_t)i * p.dim, (size_t)(i / p.heads), (int)(i % p.heads), threadIdx.x & 31);
+        return;
+    }
+    const int group = p.lanes, lane = threadIdx.x % group;
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / group;
+    const bool live = i < (long long)p.tokens * p.heads;
+    const size_t t = live ? (size_t)(i / p.heads) : 0;
+    const int at = live ? (int)(i % p.heads) * p.dim : 0;
+    const float* o = p.o_raw + t * p.heads * p.dim + at;
+    const float* g = p.proj + t * p.ldp + p.g_col + at;
+    TO* out = (TO*)p.y + t * p.ldy + at;
+    float ss = 0.f;
+    for (int d = lane * 4; d < p.dim; d += group * 4) {
+        const float4 v = *reinterpret_cast<const float4*>(o + d);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    for (int x = group >> 1; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    if (!live) return;
+    const float inv = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
+    for (int d = lane * 4; d < p.dim; d += group * 4) {
+        const float4 v = *reinterpret_cast<const float4*>(o + d), z = *reinterpret_cast<const float4*>(g + d), w = *reinterpret_cast<const float4*>(p.gain + at + d);
+        const float r0 = v.x * inv * w.x * sigmoid_f(z.x), r1 = v.y * inv * w.y * sigmoid_f(z.y), r2 = v.z * inv * w.z * sigmoid_f(z.z),
+                    r3 = v.w * inv * w.w * sigmoid_f(z.w);
+        if (sizeof(TO) == 2) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(r0, r1), hi = __floats2bfloat162_rn(r2, r3);
+            *reinterpret_cast<uint2*>(out + d) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+        } else {
+            *reinterpret_cast<float4*>(out + d) = make_float4(r0, r1, r2, r3);
+        }
+    }
 }
 
-template <typename TO, int R, int P, int COLS>
+// INLINE: the block makes its entry's records itself (entries of up to p.tile tokens)
+template <typename TO, int R, int P, bool INLINE>
 __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams p) {
-    extern __shared__ __align__(16) float smem[];
-    constexpr int RS = R + PAD, DS = RS * P;        // a part's stride, a staged vector's length (rows beyond dim hold zeros)
-    const int dim = p.dim, cols = p.cols, vcols = (cols + 3) & ~3, TILE = p.tile;
-    const int stage_floats = TILE * (VECS * DS + vcols);
-    float* s_o = smem + 2 * stage_floats;           // [TILE, cols]
+    extern __shared__ __align__(128) float smem[];
+    __shared__ __align__(8) uint64_t full[STAGES];
+    __shared__ int abort_flag;
+    constexpr int DS = R * P, REC = VECS * DS, NSTAGES = INLINE ? 1 : STAGES;
+    const int dim = p.dim, cols = p.cols, TILE = p.tile;
+    float* s_o = smem + NSTAGES * TILE * REC;       // [2][TILE][cols]
     const int head = blockIdx.x, seq = blockIdx.y, j0 = blockIdx.z * cols;
     const int start = p.seq_starts[seq], count = p.seq_starts[seq + 1] - start;
-    const int jl = threadIdx.x / P * COLS, part = threadIdx.x % P;
+    const int jl = threadIdx.x / P, part = threadIdx.x % P;
     const int width = min(cols, dim - j0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-    float* S = p.state + (size_t)p.seq_slots[seq] * p.slot_floats + p.state_offset + ((size_t)head * dim + j0 + jl) * dim + part * R;
-    float s[COLS][R];
+    const int tiles = (count + TILE - 1) / TILE;
+    const float* source = p.records + ((size_t)head * p.tokens + start) * REC;
+    auto fill = [&](int ti) {                       // one thread
+        const uint32_t bytes = (uint32_t)(min(TILE, count - ti * TILE) * REC * 4);
+        mbar_expect_tx(&full[ti % STAGES], bytes);
+        bulk_load(smem + (ti % STAGES) * TILE * REC, source + (size_t)ti * TILE * REC, bytes, &full[ti % STAGES]);
+    };
+    if (!INLINE && threadIdx.x == 0) {
+        for (int s = 0; s < STAGES; ++s) mbar_init(&full[s], 1);
+        abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+        for (int ti = 0; ti < min(STAGES - 1, tiles); ++ti) fill(ti);
+    }
+    float* S = p.state + (size_t)p.seq_slots[seq] * p.slot_floats + p.state_offset + ((size_t)head * dim + j0 + jl) * dim;
+    const bool mine = jl < width;
+    uint64_t s[R / 2];
 #pragma unroll
-    for (int c = 0; c < COLS; ++c)
-#pragma unroll
-        for (int r = 0; r < R; ++r) s[c][r] = (jl + c < width && part * R + r < dim) ? S[(size_t)c * dim + r] : 0.f;
-    for (int i = threadIdx.x; i < 2 * stage_floats; i += blockDim.x) smem[i] = 0.f;      // rows beyond dim stay zero
-    __syncthreads();
-    // vector v of a tile: [v][token][DS]; then the values [token][vcols]
-    auto fetch = [&](int ti, int b) {
-        const int t0 = ti * TILE, n = min(TILE, count - t0);
-        float* base = smem + b * stage_floats;
-        float* sv = base + VECS * TILE * DS;
-        if (p.wide) {
-            const int pieces = dim / 4;
-            for (int i = threadIdx.x; i < n * pieces; i += blockDim.x) {
-                const int t = i / pieces, d = (i % pieces) * 4;
-                const size_t tok = (size_t)(start + t0 + t);
-                const float* vec = p.vecs + (tok * p.heads + head) * 3 * dim + d;
-                const float* row = p.proj + tok * p.ldp + head * dim + d;
-                float* dst = base + t * DS + (d / R) * RS + d % R;
-                copy_async_16(dst, vec);
-                copy_async_16(dst + TILE * DS, vec + dim);
-                copy_async_16(dst + 2 * TILE * DS, vec + 2 * dim);
-                copy_async_16(dst + 3 * TILE * DS, row + p.k_col);
-                copy_async_16(dst + 4 * TILE * DS, row + p.r_col);
-            }
-            const int vp = width / 4;
-            for (int i = threadIdx.x; i < n * vp; i += blockDim.x) {
-                const int t = i / vp, d = (i % vp) * 4;
-                copy_async_16(sv + t * vcols + d, p.proj + (size_t)(start + t0 + t) * p.ldp + p.v_col + head * dim + j0 + d);
-            }
+    for (int i = 0; i < R / 4; ++i) {
+        const int row = (i * P + part) * 4;
+        float v[4];
+        if (dim % 4 == 0) {
+            const float4 f = mine && row < dim ? *reinterpret_cast<const float4*>(S + row) : make_float4(0.f, 0.f, 0.f, 0.f);
+            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
         } else {
-            for (int i = threadIdx.x; i < n * dim; i += blockDim.x) {
-                const int t = i / dim, d = i % dim;
-                const size_t tok = (size_t)(start + t0 + t);
-                const float* vec = p.vecs + (tok * p.heads + head) * 3 * dim + d;
-                const float* row = p.proj + tok * p.ldp + head * dim + d;
-                float* dst = base + t * DS + (d / R) * RS + d % R;
-                copy_async_4(dst, vec);
-                copy_async_4(dst + TILE * DS, vec + dim);
-                copy_async_4(dst + 2 * TILE * DS, vec + 2 * dim);
-                copy_async_4(dst + 3 * TILE * DS, row + p.k_col);
-                copy_async_4(dst + 4 * TILE * DS, row + p.r_col);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] = mine && row + e < dim ? S[row + e] : 0.f;
+        }
+        s[2 * i] = pair_of(v[0], v[1]);
+        s[2 * i + 1] = pair_of(v[2], v[3]);
+    }
+    if (INLINE && count > TILE) {                   // the host hands no such step here
+        if (threadIdx.x == 0) atomicOr(p.status, EG_STATUS_BAD_SLOT);
+        return;
+    }
+    if (INLINE) {
+        float* inner = s_o + 2 * TILE * cols;       // [TILE][rank]
+        for (int i = threadIdx.x; i < count * p.rank; i += blockDim.x)
+            inner[i] = tanhf(p.proj[(size_t)(start + i / p.rank) * p.ldp + p.inner_col + i % p.rank]);
+        __syncthreads();
+        // a warp per (token, 32 channels); every warp sums the whole key's squares
+        const int blocks = (DS + 31) / 32;
+        for (int it = warp; it < count * blocks; it += warps) {
+            const int t = it / blocks, d = it % blocks * 32 + lane, at = head * dim;
+            const float* row = p.proj + (size_t)(start + t) * p.ldp;
+            float kk = 0.f;
+            for (int c = lane; c < dim; c += 32) {
+                const float k = row[p.k_col + at + c];
+                kk = fmaf(k, k, kk);
             }
+            const float inv = 1.0f / sqrtf(warp_sum(kk) + p.unit_eps);
+            float* rec = smem + (size_t)t * REC;
+            if (d < dim) {
+                const TO* w2 = (const TO*)p.w2 + (size_t)(at + d) * p.ld2;
+                const float* in = inner + t * p.rank;
+                float x0 = 0.f, x1 = 0.f;
+                int r = 0;
+                if (sizeof(TO) == 2) {              // rows of w2 start on 16-byte boundaries (ld2 a multiple of 8)
+                    for (; r + 8 <= p.rank; r += 8) {
+                        const uint4 q = *reinterpret_cast<const uint4*>(w2 + r);
+                        const uint32_t m[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            x0 = fmaf(__uint_as_float(m[e] << 16), in[r + 2 * e], x0);
+                            x1 = fmaf(__uint_as_float(m[e] & 0xffff0000u), in[r + 2 * e + 1], x1);
+                        }
+                    }
+                }
+                for (; r < p.rank; ++r) x0 = fmaf(to_f32<TO>(w2[r]), in[r], x0);
+                put_channel(p, row, at, d, x0 + x1, inv, rec, DS);
+            } else if (d < DS) {
+                for (int q = 0; q < VECS; ++q) rec[q * DS + d] = 0.f;
+            }
+        }
+    }
+    __syncthreads();
+    auto write_out = [&](int ti) {                  // the outputs of tile ti, complete in s_o
+        const int t0 = ti * TILE, n = min(TILE, count - t0);
+        const float* o = s_o + (ti & 1) * TILE * cols;
+        if (p.o_raw) {
             for (int i = threadIdx.x; i < n * width; i += blockDim.x) {
                 const int t = i / width, d = i % width;
-                copy_async_4(sv + t * vcols + d, p.proj + (size_t)(start + t0 + t) * p.ldp + p.v_col + head * dim + j0 + d);
+                p.o_raw[(size_t)(start + t0 + t) * ((size_t)p.heads * dim) + head * dim + j0 + d] = o[t * cols + d];
             }
-        }
-        asm volatile("cp.async.commit_group;\n" ::: "memory");
-    };
-    const int tiles = (count + TILE - 1) / TILE;
-    if (tiles > 0) fetch(0, 0);
-    for (int ti = 0; ti < tiles; ++ti) {
-        const int t0 = ti * TILE, n = min(TILE, count - t0);
-        if (ti + 1 < tiles) {
-            fetch(ti + 1, (ti + 1) & 1);
-            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
         } else {
-            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+            for (int t = warp; t < n; t += warps) norm_and_gate<TO>(p, o + t * cols, (size_t)(start + t0 + t), head, lane);
         }
-        __syncthreads();                            // this tile has arrived; the tile before is done with s_o
-        const float* base = smem + (ti & 1) * stage_floats;
-        const float* s_v = base + VECS * TILE * DS;
+    };
+    bool ok = true;
+    int done = 0;
+    for (int ti = 0; ti < tiles; ++ti) {
+        if (!INLINE) {
+            ok = mbar_wait_bounded(&full[ti % STAGES], (ti / STAGES) & 1, &abort_flag, p.status, WAIT_LIMIT);
+            ok = __syncthreads_and(ok);             // every warp is done with the tile before: its stage may be filled again, its outputs read
+            if (!ok) break;
+            if (threadIdx.x == 0 && ti + STAGES - 1 < tiles) fill(ti + STAGES - 1);
+        } else if (ti > 0) {
+            break;                                  // entries that make their records here are one tile
+        }
+        if (ti > 0) write_out(ti - 1);
+        const int n = min(TILE, count - ti * TILE);
+        const float* base = smem + (INLINE ? 0 : ti % STAGES) * TILE * REC;
+        float* out = s_o + (ti & 1) * TILE * cols + jl;
         auto step = [&](int t) {
-            const float* at = base + t * DS + part * RS;
-            auto piece = [&](int v, int r) { return *reinterpret_cast<const float4*>(at + v * TILE * DS + r); };
+            const float* rec = base + t * REC + part * 4;
+            auto piece = [&](int v, int i) { return *reinterpret_cast<const ulonglong2*>(rec + v * DS + i * P * 4); };
             // what the old state holds along the unit key
-            float held[COLS][2] = {};
+            uint64_t held[2] = {0ull, 0ull};
 #pragma unroll
-            for (int r = 0; r < R; r += 4) {
-                const float4 u = piece(1, r);
-#pragma unroll
-                for (int c = 0; c < COLS; ++c) {
-                    held[c][0] = fmaf(s[c][r], u.x, held[c][0]);
-                    held[c][1] = fmaf(s[c][r + 1], u.y, held[c][1]);
-                    held[c][0] = fmaf(s[c][r + 2], u.z, held[c][0]);
-                    held[c][1] = fmaf(s[c][r + 3], u.w, held[c][1]);
-                }
+            for (int i = 0; i < R / 4; ++i) {
+                const ulonglong2 u = piece(1, i);
+                held[0] = fma2(s[2 * i], u.x, held[0]);
+                held[1] = fma2(s[2 * i + 1], u.y, held[1]);
             }
-            float off[COLS], value[COLS], read[COLS][2] = {};
-#pragma unroll
-            for (int c = 0; c < COLS; ++c) {
-                off[c] = held[c][0] + held[c][1];
-                value[c] = s_v[t * vcols + jl + c];
-            }
+            const float value = base[t * REC + 5 * DS + j0 + jl];
+            const uint64_t value2 = pair_of(value, value);
             // meanwhile the rows decay and take in the value
 #pragma unroll
-            for (int r = 0; r < R; r += 4) {
-                const float4 w = piece(0, r), k = piece(3, r);
-#pragma unroll
-                for (int c = 0; c < COLS; ++c) {
-                    s[c][r] = fmaf(k.x, value[c], w.x * s[c][r]);
-                    s[c][r + 1] = fmaf(k.y, value[c], w.y * s[c][r + 1]);
-                    s[c][r + 2] = fmaf(k.z, value[c], w.z * s[c][r + 2]);
-                    s[c][r + 3] = fmaf(k.w, value[c], w.w * s[c][r + 3]);
-                }
+            for (int i = 0; i < R / 4; ++i) {
+                const ulonglong2 w = piece(0, i), k = piece(3, i);
+                s[2 * i] = fma2(w.x, s[2 * i], mul2(k.x, value2));
+                s[2 * i + 1] = fma2(w.y, s[2 * i + 1], mul2(k.y, value2));
             }
+            float off = sum_of(held[0]) + sum_of(held[1]);
 #pragma unroll
-            for (int o = 1; o < P; o <<= 1)
+            for (int o = 1; o < P; o <<= 1) off += __shfl_xor_sync(0xffffffffu, off, o);
+            const uint64_t off2 = pair_of(-off, -off);
+            uint64_t read[2] = {0ull, 0ull};
 #pragma unroll
-                for (int c = 0; c < COLS; ++c) off[c] += __shfl_xor_sync(0xffffffffu, off[c], o);
-#pragma unroll
-            for (int r = 0; r < R; r += 4) {
-                const float4 a = piece(2, r), q = piece(4, r);
-#pragma unroll
-                for (int c = 0; c < COLS; ++c) {
-                    s[c][r] = fmaf(-a.x, off[c], s[c][r]);
-                    s[c][r + 1] = fmaf(-a.y, off[c], s[c][r + 1]);
-                    s[c][r + 2] = fmaf(-a.z, off[c], s[c][r + 2]);
-                    s[c][r + 3] = fmaf(-a.w, off[c], s[c][r + 3]);
-                    read[c][0] = fmaf(s[c][r], q.x, read[c][0]);
-                    read[c][1] = fmaf(s[c][r + 1], q.y, read[c][1]);
-                    read[c][0] = fmaf(s[c][r + 2], q.z, read[c][0]);
-                    read[c][1] = fmaf(s[c][r + 3], q.w, read[c][1]);
-                }
+            for (int i = 0; i < R / 4; ++i) {
+                const ulonglong2 a = piece(2, i), q = piece(4, i);
+                s[2 * i] = fma2(a.x, off2, s[2 * i]);
+                s[2 * i + 1] = fma2(a.y, off2, s[2 * i + 1]);
+                read[0] = fma2(s[2 * i], q.x, read[0]);
+                read[1] = fma2(s[2 * i + 1], q.y, read[1]);
             }
+            float o = sum_of(read[0]) + sum_of(read[1]);
 #pragma unroll
-            for (int c = 0; c < COLS; ++c) {
-                float o = read[c][0] + read[c][1];
-#pragma unroll
-                for (int x = 1; x < P; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-                if (part == 0 && jl + c < width) s_o[t * cols + jl + c] = o;
-            }
+            for (int x = 1; x < P; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
+            if (part == 0 && mine) out[t * cols] = o;
         };
-        if (n == TILE && TILE == 16) {              // a whole tile: unrolled, so that the loads of the next tokens go out ahead of their steps
+        if (!INLINE && n == 16) {                   // a whole tile: unrolled, so that the loads of the next tokens go out ahead of their steps
 #pragma unroll 4
             for (int t = 0; t < 16; ++t) step(t);
         } else {
             for (int t = 0; t < n; ++t) step(t);
         }
-        __syncthreads();                            // the tile's outputs are complete; its buffer may be filled again
-        if (p.o_raw) {
-            for (int i = threadIdx.x; i < n * width; i += blockDim.x) {
-                const int t = i / width, d = i % width;
-                p.o_raw[(size_t)(start + t0 + t) * ((size_t)p.heads * dim) + head * dim + j0 + d] = s_o[t * cols + d];
-            }
+        done = ti + 1;
+    }
+    if (!INLINE && !ok) {                           // every copy has to land before the block gives up its shared memory
+        if (threadIdx.x == 0)
+            for (int ti = done; ti < min(done + STAGES - 1, tiles); ++ti)
+                for (unsigned i = 0; i < WAIT_LIMIT && !mbar_try_wait(&full[ti % STAGES], (ti / STAGES) & 1); ++i) {}
+        return;
+    }
+    __syncthreads();
+    if (tiles > 0) write_out(INLINE ? 0 : tiles - 1);
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const int row = (i * P + part) * 4;
+        float v[4];
+        asm("mov.b64 {%0, %1}, %2;" : "=f"(v[0]), "=f"(v[1]) : "l"(s[2 * i]));
+        asm("mov.b64 {%0, %1}, %2;" : "=f"(v[2]), "=f"(v[3]) : "l"(s[2 * i + 1]));
+        if (!mine) continue;
+        if (dim % 4 == 0) {
+            if (row < dim) *reinterpret_cast<float4*>(S + row) = make_float4(v[0], v[1], v[2], v[3]);
         } else {
-            for (int t = warp; t < n; t += warps) norm_and_gate<TO>(p, s_o + t * cols, (size_t)(start + t0 + t), head, lane);
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (row + e < dim) S[row + e] = v[e];
         }
     }
-#pragma unroll
-    for (int c = 0; c < COLS; ++c)
-#pragma unroll
-        for (int r = 0; r < R; ++r)
-            if (jl + c < width && part * R + r < dim) S[(size_t)c * dim + r] = s[c][r];
 }
 
-template <typename TO, int R, int P, int COLS>
-int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num_seqs) {
-    // columns a block: whole warps of them, a multiple of four (the slices' values start on 16-byte boundaries)
-    constexpr int per_warp = 32 / P * COLS < 4 ? 4 : 32 / P * COLS;
-    const int most = 512 / P * COLS / per_warp * per_warp;
+int power_of_two_lanes(int items) {                 // the least power of two that is at least `items`, up to 32
+    int n = 1;
+    while (n < items && n < 32) n <<= 1;
+    return n;
+}
+
+template <typename TO, int R, int P, bool INLINE>
+int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num_seqs, bool float4_rows) {
+    constexpr int DS = R * P, REC = VECS * DS, per_warp = 32 / P < 1 ? 1 : 32 / P;
+    const int most = 512 / P / per_warp * per_warp;
     if (!p.o_raw) slices = 1;
     int cols = (p.dim + slices - 1) / slices;
     cols = std::min((cols + per_warp - 1) / per_warp * per_warp, most);
@@ -267,32 +399,40 @@ int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num
     if (slices > 1 && !p.o_raw) return (int)cudaErrorInvalidValue;
     if (slices == 1) p.o_raw = nullptr;
     p.cols = cols;
-    const int threads = cols / COLS * P, vcols = (cols + 3) & ~3;
-    auto bytes = [&](int tile) { return ((size_t)2 * tile * (VECS * (R + PAD) * P + vcols) + (size_t)tile * cols) * sizeof(float); };
-    p.tile = 16;
-    while (p.tile > 2 && bytes(p.tile) > 200 * 1024) p.tile /= 2;
-    const size_t smem = bytes(p.tile);
-    if (threads > 512 || smem > 200 * 1024) return (int)cudaErrorInvalidValue;
-    auto kernel = general_delta_kernel<TO, R, P, COLS>;
+    p.tile = DS <= 128 ? 16 : 8;
+    const size_t smem = ((size_t)(INLINE ? 1 : STAGES) * p.tile * REC + (size_t)2 * p.tile * cols + (INLINE ? (size_t)p.tile * p.rank : 0)) * sizeof(float);
+    if (smem > 220 * 1024) return (int)cudaErrorInvalidValue;
+    auto kernel = general_delta_kernel<TO, R, P, INLINE>;
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
-    p.wide = p.dim % 4 == 0 && p.ldp % 4 == 0 && p.r_col % 4 == 0 && p.k_col % 4 == 0 && p.v_col % 4 == 0 && (uintptr_t)p.proj % 16 == 0 && (uintptr_t)p.vecs % 16 == 0;
-    const long long warps = (long long)p.tokens * p.heads;
-    general_delta_prepare_kernel<<<(unsigned)((warps + 3) / 4), 128, 0, stream>>>(p);
-    kernel<<<dim3(p.heads, num_seqs, slices), threads, smem, stream>>>(p);
-    if (p.o_raw) general_delta_output_kernel<TO><<<(unsigned)((warps + 3) / 4), 128, 0, stream>>>(p);
+    const bool wide = float4_rows && p.dim % 4 == 0;
+    if (!INLINE) {
+        p.lanes = power_of_two_lanes(wide ? DS / 4 : DS);
+        const unsigned blocks = (unsigned)(((long long)p.tokens * p.heads * p.lanes + 255) / 256);
+        if (wide) general_delta_records_kernel<true><<<blocks, 256, 0, stream>>>(p, DS);
+        else general_delta_records_kernel<false><<<blocks, 256, 0, stream>>>(p, DS);
+    }
+    kernel<<<dim3(p.heads, num_seqs, slices), cols * P, smem, stream>>>(p);
+    if (p.o_raw) {
+        if (wide) {
+            p.lanes = power_of_two_lanes((p.dim + 3) / 4);
+            general_delta_output_kernel<TO, true><<<(unsigned)(((long long)p.tokens * p.heads * p.lanes + 255) / 256), 256, 0, stream>>>(p);
+        } else {
+            general_delta_output_kernel<TO, false><<<(unsigned)(((long long)p.tokens * p.heads + 7) / 8), 256, 0, stream>>>(p);
+        }
+    }
     return eg_launch_status();
 }
 
-template <typename TO>
-int dispatch_general_delta(cudaStream_t stream, const DeltaParams& p, int slices, int num_seqs) {
-    if (p.dim <= 16) return launch_general_delta<TO, 4, 4, 1>(stream, p, slices, num_seqs);
-    if (p.dim <= 32) return launch_general_delta<TO, 8, 4, 1>(stream, p, slices, num_seqs);
-    if (p.dim <= 64) return launch_general_delta<TO, 8, 8, 2>(stream, p, slices, num_seqs);
-    if (p.dim <= 128) return launch_general_delta<TO, 8, 16, 2>(stream, p, slices, num_seqs);
-    return launch_general_delta<TO, 8, 32, 2>(stream, p, slices, num_seqs);
+template <typename TO, bool INLINE>
+int dispatch_general_delta(cudaStream_t stream, const DeltaParams& p, int slices, int num_seqs, bool wide) {
+    if (p.dim <= 16) return launch_general_delta<TO, 4, 4, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 32) return launch_general_delta<TO, 8, 4, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 64) return launch_general_delta<TO, 16, 4, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 128) return launch_general_delta<TO, 16, 8, INLINE>(stream, p, slices, num_seqs, wide);
+    return launch_general_delta<TO, 16, 16, INLINE>(stream, p, slices, num_seqs, wide);
 }
 
 template <typename T>
@@ -304,17 +444,28 @@ __global__ void tanh_columns_kernel(const float* __restrict__ src, long long lds
 }
 }  // namespace
 
+// float32 values of a record of a head of `dim` channels (scratch: heads * tokens of them)
+EG_API int eg_general_delta_record(int dim) { return VECS * (dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256); }
+
+// up to how many tokens an entry may have, and how large the inner size may be, for eg_general_delta with x null
+EG_API int eg_general_delta_inline_takes(int entry_tokens, int rank) { return entry_tokens <= 8 && rank <= 512; }
+
 // proj float32 [tokens, ldp] with r, k, v, g (the output gate) and a (the removal rates' logits, bias a0 still to be added), heads x dim
-// each, at their columns; x float32 [tokens, ldx]: the decays' logits (w0 still to be added); a0, w0, gain float32 [heads * dim].
-// vecs float32 [tokens, heads, 3, dim] of scratch.  state: the requests' slots; S of a request lies state_offset floats into its
-// slot.  y [tokens, ldy] in y_dtype.  slices > 1 (with o_raw float32 [tokens, heads * dim]): a head's columns are dealt to that many
-// blocks, and the outputs are normed by a kernel behind.  dim up to 256.
-EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ldp, int r_col, int k_col, int v_col, int g_col, int a_col, const float* x,
-                            long long ldx, const float* w0, const float* a0, const float* gain, float* vecs, float* state, long long slot_floats,
-                            long long state_offset, const int* seq_starts, const int* seq_slots, void* y, int y_dtype, long long ldy, float* o_raw, int slices,
-                            int tokens, int num_seqs, int heads, int dim, float unit_eps, float eps, float decay_scale) {
+// each, and the inner values of the decays' map (before tanh, `rank`) at their columns; x float32 [tokens, ldx]: the decays' logits
+// (w0 still to be added), or null in steps whose entries eg_general_delta_inline_takes: then w2 [heads * dim, ld2] in y_dtype (ld2 a
+// multiple of 8).  a0, w0, gain float32 [heads * dim].  records: scratch, not read with x null.  state: the requests' slots; S of
+// a request lies state_offset floats into its slot.  y [tokens, ldy] in y_dtype.  slices > 1 (with o_raw float32 [tokens, heads * dim]): a
+// head's columns are dealt to that many blocks, and the outputs are normed by a kernel behind.  dim up to 256.
+EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ldp, int r_col, int k_col, int v_col, int g_col, int a_col, int inner_col,
+                            const float* x, long long ldx, const void* w2, int ld2, int rank, const float* w0, const float* a0, const float* gain,
+                            float* records, float* state, long long slot_floats, long long state_offset, const int* seq_starts, const int* seq_slots,
+                            void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps,
+                            float eps, float decay_scale, int* status) {
     if (num_seqs <= 0 || tokens <= 0) return 0;
-    if (heads <= 0 || dim <= 0 || dim > 256 || slices < 1 || !vecs) return (int)cudaErrorInvalidValue;
+    if (heads <= 0 || dim <= 0 || dim > 256 || slices < 1 || (x && !records) || (!x && (!w2 || ld2 % 8 || (uintptr_t)w2 % 16))) return (int)cudaErrorInvalidValue;
+    if (slot_floats % 4 || state_offset % 4 || (uintptr_t)state % 16 || (uintptr_t)records % 16) {
+        if (dim % 4 == 0 || (uintptr_t)records % 16) return (int)cudaErrorInvalidValue;     // heads of a multiple of four rows are read in 16-byte pieces
+    }
     DeltaParams p{};
     p.proj = proj;
     p.ldp = ldp;
@@ -323,12 +474,16 @@ EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ld
     p.v_col = v_col;
     p.g_col = g_col;
     p.a_col = a_col;
+    p.inner_col = inner_col;
     p.x = x;
     p.ldx = ldx;
+    p.w2 = w2;
+    p.ld2 = ld2;
+    p.rank = rank;
     p.w0 = w0;
     p.a0 = a0;
     p.gain = gain;
-    p.vecs = vecs;
+    p.records = records;
     p.state = state;
     p.slot_floats = slot_floats;
     p.state_offset = state_offset;
@@ -343,7 +498,13 @@ EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ld
     p.unit_eps = unit_eps;
     p.eps = eps;
     p.decay_scale = decay_scale;
-    return y_dtype == EG_BF16 ? dispatch_general_delta<bf16>(stream, p, slices, num_seqs) : dispatch_general_delta<float>(stream, p, slices, num_seqs);
+    p.status = status;
+    auto aligned = [](const void* q) { return (uintptr_t)q % 16 == 0; };
+    const bool wide = ldp % 4 == 0 && ldx % 4 == 0 && r_col % 4 == 0 && k_col % 4 == 0 && v_col % 4 == 0 && g_col % 4 == 0 && a_col % 4 == 0 && aligned(proj) &&
+                      aligned(x) && aligned(w0) && aligned(a0) && aligned(gain) && aligned(o_raw) && aligned(y) && ldy % 4 == 0;
+    if (y_dtype == EG_BF16)
+        return x ? dispatch_general_delta<bf16, false>(stream, p, slices, num_seqs, wide) : dispatch_general_delta<bf16, true>(stream, p, slices, num_seqs, wide);
+    return x ? dispatch_general_delta<float, false>(stream, p, slices, num_seqs, wide) : dispatch_general_delta<float, true>(stream, p, slices, num_seqs, wide);
 }
 
 // dst [rows, ldd] in dst_dtype: column c < cols holds tanh(src[., c]), columns up to `padded` hold zeros
