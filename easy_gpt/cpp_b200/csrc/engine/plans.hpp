@@ -185,13 +185,12 @@ inline int delta_column_slices(int entries, int heads, int value_dim) {
     return (int)std::max<long long>(1, std::min<long long>(wanted, value_dim / 8));
 }
 
-// The same for the generalised delta rule, whose step is bound by the latency of one token's chain: a warp runs as fast as it can
-// while it has an SM sub-core to itself, so a block has four warps (32, 16 or 8 columns of heads of up to 64, 128, 256 rows)
-// while the step has few (entry, head) pairs, and whole heads where these fill the SMs.
+// The same for the generalised delta rule: as many blocks as there are SMs, of at least one warp (8 columns; 4 of heads of more
+// than 128 rows).  Its warps read every token's vectors out of shared memory, whose rate is what several warps of an SM share.
 inline int general_delta_slices(int entries, int heads, int dim) {
     const long long blocks = (long long)std::max(1, entries) * heads;
-    const int columns = dim <= 64 ? 32 : dim <= 128 ? 16 : 8;
-    return (int)std::max<long long>(1, std::min<long long>((dim + columns - 1) / columns, (sm_count() + blocks - 1) / blocks));
+    const int columns = dim <= 128 ? 8 : 4;
+    return (int)std::max<long long>(1, std::min<long long>((dim + columns - 1) / columns, sm_count() / blocks));
 }
 
 inline int scan_states_per_lane(int channels, int states) {

@@ -14,11 +14,13 @@
 // them (a group of lanes per token and head).  In steps whose entries are a few tokens each (decoding) the recurrence's own blocks make
 // them in shared memory, and work out x as well (W_2 is small), which saves two kernels and a product.
 //
-// Recurrence: one block per (head, batch entry, slice of the head's columns: the columns of S do not depend on one another).  A
-// column of S belongs to P neighbouring lanes, each with R of its rows in registers for the entry's whole run of tokens (lane p
-// has rows 4 (i P + p) .. + 3: neighbouring lanes read neighbouring 16-byte pieces).  Per token the dot product with u over the old
-// rows is the only thing the next token waits for: R/4 dependent multiply-adds and log2 P shuffles; decay, value and the dot
-// product with r run beside them, all on pairs of float32.  Tiles arrive three stages ahead.  Outputs are normed and gated by the
+// Recurrence: one block per (head, batch entry, slice of the head's columns: the columns of S do not depend on one another).  COLS
+// neighbouring columns of S belong to P neighbouring lanes, each with R of their rows in registers for the entry's whole run of
+// tokens (lane p has rows 4 (i P + p) .. + 3: eight neighbouring lanes read 128 neighbouring bytes, what shared memory hands out at a
+// time).  Per token the dot product with u over the old rows is the only thing the next token waits for: R/4 dependent multiply-adds
+// and log2 P shuffles; decay, value and the dot product with r run beside them, all on pairs of float32.  (Measured on B200, 32 heads
+// of 64: with one column a thread, P = 4 and R = 16 a token took 516 cycles: every warp reads all five vectors for its columns, and
+// shared memory hands out four times the bytes that differ.)  Tiles arrive three stages ahead.  Outputs are normed and gated by the
 // block where it holds a whole head, else by a kernel behind.  The slot keeps S as [head, column, row].  The order of every sum
 // depends on the sizes alone.
 #include <algorithm>
@@ -196,7 +198,7 @@ __global__ void __launch_bounds__(256) general_delta_output_kernel(const DeltaPa
 }
 
 // INLINE: the block makes its entry's records itself (entries of up to p.tile tokens)
-template <typename TO, int R, int P, bool INLINE>
+template <typename TO, int R, int P, int COLS, bool INLINE>
 __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams p) {
     extern __shared__ __align__(128) float smem[];
     __shared__ __align__(8) uint64_t full[STAGES];
@@ -206,7 +208,7 @@ __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams
     float* s_o = smem + NSTAGES * TILE * REC;       // [2][TILE][cols]
     const int head = blockIdx.x, seq = blockIdx.y, j0 = blockIdx.z * cols;
     const int start = p.seq_starts[seq], count = p.seq_starts[seq + 1] - start;
-    const int jl = threadIdx.x / P, part = threadIdx.x % P;
+    const int jl = threadIdx.x / P * COLS, part = threadIdx.x % P;
     const int width = min(cols, dim - j0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int tiles = (count + TILE - 1) / TILE;
@@ -223,22 +225,25 @@ __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams
         for (int ti = 0; ti < min(STAGES - 1, tiles); ++ti) fill(ti);
     }
     float* S = p.state + (size_t)p.seq_slots[seq] * p.slot_floats + p.state_offset + ((size_t)head * dim + j0 + jl) * dim;
-    const bool mine = jl < width;
-    uint64_t s[R / 2];
+    uint64_t s[COLS][R / 2];
 #pragma unroll
-    for (int i = 0; i < R / 4; ++i) {
-        const int row = (i * P + part) * 4;
-        float v[4];
-        if (dim % 4 == 0) {
-            const float4 f = mine && row < dim ? *reinterpret_cast<const float4*>(S + row) : make_float4(0.f, 0.f, 0.f, 0.f);
-            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-        } else {
+    for (int c = 0; c < COLS; ++c)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) v[e] = mine && row + e < dim ? S[row + e] : 0.f;
+        for (int i = 0; i < R / 4; ++i) {
+            const int row = (i * P + part) * 4;
+            const float* at = S + (size_t)c * dim + row;
+            const bool mine = jl + c < width;
+            float v[4];
+            if (dim % 4 == 0) {
+                const float4 f = mine && row < dim ? *reinterpret_cast<const float4*>(at) : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v[e] = mine && row + e < dim ? at[e] : 0.f;
+            }
+            s[c][2 * i] = pair_of(v[0], v[1]);
+            s[c][2 * i + 1] = pair_of(v[2], v[3]);
         }
-        s[2 * i] = pair_of(v[0], v[1]);
-        s[2 * i + 1] = pair_of(v[2], v[3]);
-    }
     if (INLINE && count > TILE) {                   // the host hands no such step here
         if (threadIdx.x == 0) atomicOr(p.status, EG_STATUS_BAD_SLOT);
         return;
@@ -315,39 +320,73 @@ __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams
             const float* rec = base + t * REC + part * 4;
             auto piece = [&](int v, int i) { return *reinterpret_cast<const ulonglong2*>(rec + v * DS + i * P * 4); };
             // what the old state holds along the unit key
-            uint64_t held[2] = {0ull, 0ull};
+            uint64_t held[COLS][2] = {};
 #pragma unroll
             for (int i = 0; i < R / 4; ++i) {
                 const ulonglong2 u = piece(1, i);
-                held[0] = fma2(s[2 * i], u.x, held[0]);
-                held[1] = fma2(s[2 * i + 1], u.y, held[1]);
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) {
+                    held[c][0] = fma2(s[c][2 * i], u.x, held[c][0]);
+                    held[c][1] = fma2(s[c][2 * i + 1], u.y, held[c][1]);
+                }
             }
-            const float value = base[t * REC + 5 * DS + j0 + jl];
-            const uint64_t value2 = pair_of(value, value);
+            float off[COLS];
+            uint64_t value2[COLS];
+#pragma unroll
+            for (int c = 0; c < COLS; ++c) {
+                off[c] = sum_of(held[c][0]) + sum_of(held[c][1]);
+                const float value = base[t * REC + 5 * DS + j0 + jl + c];
+                value2[c] = pair_of(value, value);
+            }
             // meanwhile the rows decay and take in the value
 #pragma unroll
             for (int i = 0; i < R / 4; ++i) {
                 const ulonglong2 w = piece(0, i), k = piece(3, i);
-                s[2 * i] = fma2(w.x, s[2 * i], mul2(k.x, value2));
-                s[2 * i + 1] = fma2(w.y, s[2 * i + 1], mul2(k.y, value2));
-            }
-            float off = sum_of(held[0]) + sum_of(held[1]);
 #pragma unroll
-            for (int o = 1; o < P; o <<= 1) off += __shfl_xor_sync(0xffffffffu, off, o);
-            const uint64_t off2 = pair_of(-off, -off);
-            uint64_t read[2] = {0ull, 0ull};
+                for (int c = 0; c < COLS; ++c) {
+                    s[c][2 * i] = fma2(w.x, s[c][2 * i], mul2(k.x, value2[c]));
+                    s[c][2 * i + 1] = fma2(w.y, s[c][2 * i + 1], mul2(k.y, value2[c]));
+                }
+            }
+#pragma unroll
+            for (int o = 1; o < P; o <<= 1)
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) off[c] += __shfl_xor_sync(0xffffffffu, off[c], o);
+            uint64_t off2[COLS], read[COLS][2] = {};
+#pragma unroll
+            for (int c = 0; c < COLS; ++c) off2[c] = pair_of(-off[c], -off[c]);
 #pragma unroll
             for (int i = 0; i < R / 4; ++i) {
                 const ulonglong2 a = piece(2, i), q = piece(4, i);
-                s[2 * i] = fma2(a.x, off2, s[2 * i]);
-                s[2 * i + 1] = fma2(a.y, off2, s[2 * i + 1]);
-                read[0] = fma2(s[2 * i], q.x, read[0]);
-                read[1] = fma2(s[2 * i + 1], q.y, read[1]);
-            }
-            float o = sum_of(read[0]) + sum_of(read[1]);
 #pragma unroll
-            for (int x = 1; x < P; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-            if (part == 0 && mine) out[t * cols] = o;
+                for (int c = 0; c < COLS; ++c) {
+                    s[c][2 * i] = fma2(a.x, off2[c], s[c][2 * i]);
+                    s[c][2 * i + 1] = fma2(a.y, off2[c], s[c][2 * i + 1]);
+                    read[c][0] = fma2(s[c][2 * i], q.x, read[c][0]);
+                    read[c][1] = fma2(s[c][2 * i + 1], q.y, read[c][1]);
+                }
+            }
+            float o[COLS];
+#pragma unroll
+            for (int c = 0; c < COLS; ++c) o[c] = sum_of(read[c][0]) + sum_of(read[c][1]);
+            // the columns' sums over the lanes: while a lane has several columns it gives half of them away for the other half
+            int col = 0;
+#pragma unroll
+            for (int x = 1, have = COLS; x < P; x <<= 1) {
+                if (have > 1) {
+                    have >>= 1;
+                    const bool upper = part & x;
+#pragma unroll
+                    for (int c = 0; c < have; ++c) {
+                        const float give = upper ? o[c] : o[have + c], keep = upper ? o[have + c] : o[c];
+                        o[c] = keep + __shfl_xor_sync(0xffffffffu, give, x);
+                    }
+                    col += upper ? have : 0;
+                } else {
+                    o[0] += __shfl_xor_sync(0xffffffffu, o[0], x);
+                }
+            }
+            if (part < COLS && jl + col < width) out[t * cols + col] = o[0];
         };
         if (!INLINE && n == 16) {                   // a whole tile: unrolled, so that the loads of the next tokens go out ahead of their steps
 #pragma unroll 4
@@ -366,20 +405,23 @@ __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams
     __syncthreads();
     if (tiles > 0) write_out(INLINE ? 0 : tiles - 1);
 #pragma unroll
-    for (int i = 0; i < R / 4; ++i) {
-        const int row = (i * P + part) * 4;
-        float v[4];
-        asm("mov.b64 {%0, %1}, %2;" : "=f"(v[0]), "=f"(v[1]) : "l"(s[2 * i]));
-        asm("mov.b64 {%0, %1}, %2;" : "=f"(v[2]), "=f"(v[3]) : "l"(s[2 * i + 1]));
-        if (!mine) continue;
-        if (dim % 4 == 0) {
-            if (row < dim) *reinterpret_cast<float4*>(S + row) = make_float4(v[0], v[1], v[2], v[3]);
-        } else {
+    for (int c = 0; c < COLS; ++c)
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
-                if (row + e < dim) S[row + e] = v[e];
+        for (int i = 0; i < R / 4; ++i) {
+            const int row = (i * P + part) * 4;
+            float* at = S + (size_t)c * dim + row;
+            float v[4];
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(v[0]), "=f"(v[1]) : "l"(s[c][2 * i]));
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(v[2]), "=f"(v[3]) : "l"(s[c][2 * i + 1]));
+            if (jl + c >= width) continue;
+            if (dim % 4 == 0) {
+                if (row < dim) *reinterpret_cast<float4*>(at) = make_float4(v[0], v[1], v[2], v[3]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (row + e < dim) at[e] = v[e];
+            }
         }
-    }
 }
 
 int power_of_two_lanes(int items) {                 // the least power of two that is at least `items`, up to 32
@@ -388,10 +430,11 @@ int power_of_two_lanes(int items) {                 // the least power of two th
     return n;
 }
 
-template <typename TO, int R, int P, bool INLINE>
+template <typename TO, int R, int P, int COLS, bool INLINE>
 int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num_seqs, bool float4_rows) {
-    constexpr int DS = R * P, REC = VECS * DS, per_warp = 32 / P < 1 ? 1 : 32 / P;
-    const int most = 512 / P / per_warp * per_warp;
+    constexpr int DS = R * P, REC = VECS * DS, per_warp = 32 / P * COLS;
+    static_assert(COLS <= P, "a lane ends with one column's sum");
+    const int most = 512 / P * COLS / per_warp * per_warp;
     if (!p.o_raw) slices = 1;
     int cols = (p.dim + slices - 1) / slices;
     cols = std::min((cols + per_warp - 1) / per_warp * per_warp, most);
@@ -402,7 +445,7 @@ int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num
     p.tile = DS <= 128 ? 16 : 8;
     const size_t smem = ((size_t)(INLINE ? 1 : STAGES) * p.tile * REC + (size_t)2 * p.tile * cols + (INLINE ? (size_t)p.tile * p.rank : 0)) * sizeof(float);
     if (smem > 220 * 1024) return (int)cudaErrorInvalidValue;
-    auto kernel = general_delta_kernel<TO, R, P, INLINE>;
+    auto kernel = general_delta_kernel<TO, R, P, COLS, INLINE>;
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
@@ -414,7 +457,7 @@ int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num
         if (wide) general_delta_records_kernel<true><<<blocks, 256, 0, stream>>>(p, DS);
         else general_delta_records_kernel<false><<<blocks, 256, 0, stream>>>(p, DS);
     }
-    kernel<<<dim3(p.heads, num_seqs, slices), cols * P, smem, stream>>>(p);
+    kernel<<<dim3(p.heads, num_seqs, slices), cols / COLS * P, smem, stream>>>(p);
     if (p.o_raw) {
         if (wide) {
             p.lanes = power_of_two_lanes((p.dim + 3) / 4);
@@ -428,11 +471,11 @@ int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num
 
 template <typename TO, bool INLINE>
 int dispatch_general_delta(cudaStream_t stream, const DeltaParams& p, int slices, int num_seqs, bool wide) {
-    if (p.dim <= 16) return launch_general_delta<TO, 4, 4, INLINE>(stream, p, slices, num_seqs, wide);
-    if (p.dim <= 32) return launch_general_delta<TO, 8, 4, INLINE>(stream, p, slices, num_seqs, wide);
-    if (p.dim <= 64) return launch_general_delta<TO, 16, 4, INLINE>(stream, p, slices, num_seqs, wide);
-    if (p.dim <= 128) return launch_general_delta<TO, 16, 8, INLINE>(stream, p, slices, num_seqs, wide);
-    return launch_general_delta<TO, 16, 16, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 16) return launch_general_delta<TO, 4, 4, 1, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 32) return launch_general_delta<TO, 4, 8, 2, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 64) return launch_general_delta<TO, 8, 8, 2, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 128) return launch_general_delta<TO, 8, 16, 4, INLINE>(stream, p, slices, num_seqs, wide);
+    return launch_general_delta<TO, 8, 32, 4, INLINE>(stream, p, slices, num_seqs, wide);
 }
 
 template <typename T>
