@@ -199,7 +199,7 @@ __global__ void __launch_bounds__(256) general_delta_output_kernel(const DeltaPa
 
 // INLINE: the block makes its entry's records itself (entries of up to p.tile tokens)
 template <typename TO, int R, int P, int COLS, bool INLINE>
-__global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams p) {
+__global__ void __launch_bounds__(INLINE ? 512 : 256, 1) general_delta_kernel(const DeltaParams p) {
     extern __shared__ __align__(128) float smem[];
     __shared__ __align__(8) uint64_t full[STAGES];
     __shared__ int abort_flag;
@@ -316,7 +316,8 @@ __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams
         const int n = min(TILE, count - ti * TILE);
         const float* base = smem + (INLINE ? 0 : ti % STAGES) * TILE * REC;
         float* out = s_o + (ti & 1) * TILE * cols + jl;
-        auto step = [&](int t) {
+        // one token: the rows move on; o: this lane's share of the columns' outputs
+        auto step = [&](int t, float (&o)[COLS]) {
             const float* rec = base + t * REC + part * 4;
             auto piece = [&](int v, int i) { return *reinterpret_cast<const ulonglong2*>(rec + v * DS + i * P * 4); };
             // what the old state holds along the unit key
@@ -366,33 +367,41 @@ __global__ void __launch_bounds__(512, 1) general_delta_kernel(const DeltaParams
                     read[c][1] = fma2(s[c][2 * i + 1], q.y, read[c][1]);
                 }
             }
-            float o[COLS];
 #pragma unroll
             for (int c = 0; c < COLS; ++c) o[c] = sum_of(read[c][0]) + sum_of(read[c][1]);
-            // the columns' sums over the lanes: while a lane has several columns it gives half of them away for the other half
-            int col = 0;
-#pragma unroll
-            for (int x = 1, have = COLS; x < P; x <<= 1) {
-                if (have > 1) {
-                    have >>= 1;
-                    const bool upper = part & x;
-#pragma unroll
-                    for (int c = 0; c < have; ++c) {
-                        const float give = upper ? o[c] : o[have + c], keep = upper ? o[have + c] : o[c];
-                        o[c] = keep + __shfl_xor_sync(0xffffffffu, give, x);
-                    }
-                    col += upper ? have : 0;
-                } else {
-                    o[0] += __shfl_xor_sync(0xffffffffu, o[0], x);
-                }
-            }
-            if (part < COLS && jl + col < width) out[t * cols + col] = o[0];
         };
-        if (!INLINE && n == 16) {                   // a whole tile: unrolled, so that the loads of the next tokens go out ahead of their steps
-#pragma unroll 4
-            for (int t = 0; t < 16; ++t) step(t);
-        } else {
-            for (int t = 0; t < n; ++t) step(t);
+        // The outputs of G = P / COLS tokens are P sums over P lanes: in every round a lane gives half of its sums away for the other half
+        // of a neighbour's, and ends with one of them.  Until then no shared memory is written, so that the loads of the group's tokens
+        // go out ahead of their steps.  (With a sum and a store after every token the loads of a token waited for the token before
+        // it: 445 cycles a token.)
+        constexpr int G = P / COLS;
+        int t = 0;
+        for (; !INLINE && t + G <= n; t += G) {
+            float o[P];
+#pragma unroll
+            for (int i = 0; i < G; ++i) step(t + i, *reinterpret_cast<float (*)[COLS]>(&o[i * COLS]));
+            int which = 0;
+#pragma unroll
+            for (int x = 1, have = P / 2; x < P; x <<= 1, have >>= 1) {
+                const bool upper = part & x;
+#pragma unroll
+                for (int i = 0; i < have; ++i) {
+                    const float give = upper ? o[i] : o[have + i], keep = upper ? o[have + i] : o[i];
+                    o[i] = keep + __shfl_xor_sync(0xffffffffu, give, x);
+                }
+                which += upper ? have : 0;
+            }
+            if (jl + which % COLS < width) out[(t + which / COLS) * cols + which % COLS] = o[0];
+        }
+        for (; t < n; ++t) {
+            float o[COLS];
+            step(t, o);
+#pragma unroll
+            for (int c = 0; c < COLS; ++c) {
+#pragma unroll
+                for (int x = 1; x < P; x <<= 1) o[c] += __shfl_xor_sync(0xffffffffu, o[c], x);
+                if (part == 0 && jl + c < width) out[t * cols + c] = o[c];
+            }
         }
         done = ti + 1;
     }
@@ -434,7 +443,7 @@ template <typename TO, int R, int P, int COLS, bool INLINE>
 int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num_seqs, bool float4_rows) {
     constexpr int DS = R * P, REC = VECS * DS, per_warp = 32 / P * COLS;
     static_assert(COLS <= P, "a lane ends with one column's sum");
-    const int most = 512 / P * COLS / per_warp * per_warp;
+    const int most = (INLINE ? 512 : 256) / P * COLS / per_warp * per_warp;
     if (!p.o_raw) slices = 1;
     int cols = (p.dim + slices - 1) / slices;
     cols = std::min((cols + per_warp - 1) / per_warp * per_warp, most);
