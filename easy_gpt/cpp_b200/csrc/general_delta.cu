@@ -10,19 +10,28 @@
 // r, k, v, y and g are columns of one projection's float32 output; x = W_2 tanh(the projection's last columns).
 //
 // The recurrence reads a *record* per token and head: the six vectors w, u, a u, k, r, v, each filled up with zeros to DS = R * P
-// values.  Records of a head lie one behind the other, so that a tile of tokens is ONE bulk copy; a kernel over all tokens makes
-// them (a group of lanes per token and head).  In steps whose entries are a few tokens each (decoding) the recurrence's own blocks make
-// them in shared memory, and work out x as well (W_2 is small), which saves two kernels and a product.
+// values, and eight numbers.  Records of a head lie one behind the other, so that a tile of tokens is ONE bulk copy; a kernel over
+// all tokens makes them.  In steps whose entries are a few tokens each (decoding) the recurrence's own blocks make them in shared
+// memory, and work out x as well (W_2 is small), which saves two kernels and a product.
 //
 // Recurrence: one block per (head, batch entry, slice of the head's columns: the columns of S do not depend on one another).  COLS
 // neighbouring columns of S belong to P neighbouring lanes, each with R of their rows in registers for the entry's whole run of
 // tokens (lane p has rows 4 (i P + p) .. + 3: eight neighbouring lanes read 128 neighbouring bytes, what shared memory hands out at a
-// time).  Per token the dot product with u over the old rows is the only thing the next token waits for: R/4 dependent multiply-adds
-// and log2 P shuffles; decay, value and the dot product with r run beside them, all on pairs of float32.  (Measured on B200, 32 heads
-// of 64: with one column a thread, P = 4 and R = 16 a token took 516 cycles: every warp reads all five vectors for its columns, and
-// shared memory hands out four times the bytes that differ.)  Tiles arrive three stages ahead.  Outputs are normed and gated by the
-// block where it holds a whole head, else by a kernel behind.  The slot keeps S as [head, column, row].  The order of every sum
-// depends on the sizes alone.
+// time).  All arithmetic on the rows is on pairs of float32.
+//
+// A token waits for the token before it through what the state holds along its key, h = S^T u: a dot product over the rows and log2 P
+// shuffles.  So tokens go in blocks of four (counted from the entry's first token of the step), whose h all come from the state in
+// front of the block: with w_i, u_i, ... the block's vectors and W_ij = w_(j+1) .. w_(i-1) channel by channel,
+//   h_i = (u_i w_0 .. w_(i-1)) . S - sum_{j<i} (u_i . W_ij a_j u_j) h_j + sum_{j<i} (u_i . W_ij k_j) v_j
+// (nothing is divided by a decay).  The record of a block's token i holds u_i w_0 .. w_(i-1) in place of u_i, and the dot products of the
+// two sums; four dot products over the rows share their shuffle rounds, and the block's sums are a handful of multiply-adds.  The
+// up to three tokens behind the last whole block go one by one.  (Measured on B200, 32 heads of 64, cycles a token: one column a
+// thread and P = 4, 516: every warp reads all five vectors for its columns, and shared memory hands out four times the bytes that
+// differ; two columns and P = 8, 445; with the outputs of four tokens summed over the lanes together, so that the loads of a token
+// do not wait for the stores of the token before, 345; one column a thread, so twice the warps, 302.)
+//
+// Tiles arrive three stages ahead.  Outputs are normed and gated by the block where it holds a whole head, else by a kernel behind.
+// The slot keeps S as [head, column, row].  The order of every sum depends on the sizes and on a token's place in its block.
 #include <algorithm>
 #include <cstdlib>
 
@@ -33,6 +42,7 @@
 namespace {
 
 constexpr int VECS = 6, STAGES = 3;
+constexpr int BLOCK = 4, NUMBERS = 8;       // tokens of a block; a record's numbers behind its vectors: the factors of h_0..h_2, 0, of v_0..v_2, 0
 constexpr unsigned WAIT_LIMIT = 1u << 24;
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
@@ -70,10 +80,10 @@ struct DeltaParams {
     const void* w2;             // [heads * dim, ld2] in w2's dtype
     int ld2, rank;
     const float *w0, *a0, *gain;
-    float* records;             // [heads, tokens, VECS, DS]
+    float* records;             // [heads, tokens, VECS * DS + NUMBERS]
     float* state;
     long long slot_floats, state_offset;
-    const int *seq_starts, *seq_slots;
+    const int *token_seq, *seq_starts, *seq_slots;
     void* y;
     long long ldy;
     float* o_raw;               // [tokens, heads * dim], or null: the block holds whole heads
@@ -93,58 +103,98 @@ __device__ __forceinline__ void put_channel(const DeltaParams& p, const float* r
     rec[5 * DS + d] = row[p.v_col + at + d];
 }
 
-// `lanes` (a power of two up to 32) neighbouring lanes make the record of a (head, token).  WIDE: four channels a lane and pass, by
-// 16-byte loads and stores.
-template <bool WIDE>
+// `lanes` (a power of two up to 32) neighbouring lanes make the records of a block of tokens of a head: the group of the block's first
+// token does, the others have nothing to do.  A lane has CH runs of four channels; WIDE: by 16-byte loads.
+template <int CH, bool WIDE>
 __global__ void __launch_bounds__(256) general_delta_records_kernel(const DeltaParams p, int DS) {
     const int group = p.lanes, lane = threadIdx.x % group;
     const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / group;
-    const bool live = i < (long long)p.tokens * p.heads;
+    if (i >= (long long)p.tokens * p.heads) return;
     // neighbouring groups take neighbouring heads of a token: the projection's rows are read in order
-    const int t = live ? (int)(i / p.heads) : 0, h = live ? (int)(i % p.heads) : 0, at = h * p.dim;
-    const float* row = p.proj + (size_t)t * p.ldp;
-    float* rec = p.records + ((size_t)h * p.tokens + t) * VECS * DS;
-    float kk = 0.f;
-    if (WIDE) {
-        for (int d = lane * 4; d < p.dim; d += group * 4) {
-            const float4 k = *reinterpret_cast<const float4*>(row + p.k_col + at + d);
-            kk += k.x * k.x + k.y * k.y + k.z * k.z + k.w * k.w;
-        }
-    } else {
-        for (int d = lane; d < p.dim; d += group) {
-            const float k = row[p.k_col + at + d];
-            kk = fmaf(k, k, kk);
-        }
-    }
-    for (int o = group >> 1; o > 0; o >>= 1) kk += __shfl_xor_sync(0xffffffffu, kk, o);
-    if (!live) return;
-    const float inv = 1.0f / sqrtf(kk + p.unit_eps);
-    if (WIDE) {
-        for (int d = lane * 4; d < DS; d += group * 4) {
-            float4 v[VECS];
-            if (d < p.dim) {
-                auto load = [&](const float* src) { return *reinterpret_cast<const float4*>(src + at + d); };
-                const float4 x = load(p.x + (size_t)t * p.ldx), w0 = load(p.w0), a = load(row + p.a_col), a0 = load(p.a0);
-                v[3] = load(row + p.k_col);
-                v[4] = load(row + p.r_col);
-                v[5] = load(row + p.v_col);
-                auto decay = [&](float l) { return decay_exp(-p.decay_scale * sigmoid_f(l)); };
-                v[0] = make_float4(decay(x.x + w0.x), decay(x.y + w0.y), decay(x.z + w0.z), decay(x.w + w0.w));
-                v[1] = make_float4(v[3].x * inv, v[3].y * inv, v[3].z * inv, v[3].w * inv);
-                v[2] = make_float4(sigmoid_f(a.x + a0.x) * v[1].x, sigmoid_f(a.y + a0.y) * v[1].y, sigmoid_f(a.z + a0.z) * v[1].z, sigmoid_f(a.w + a0.w) * v[1].w);
-            } else {
+    const int t = (int)(i / p.heads), h = (int)(i % p.heads), at = h * p.dim;
+    const int seq = p.token_seq[t], start = p.seq_starts[seq], left = p.seq_starts[seq + 1] - t;
+    if ((t - start) % BLOCK) return;
+    const unsigned mask = group == 32 ? 0xffffffffu : ((1u << group) - 1u) << (threadIdx.x % 32 / group * group);
+    auto over_group = [&](float v) {
+        for (int o = group >> 1; o > 0; o >>= 1) v += __shfl_xor_sync(mask, v, o);
+        return v;
+    };
+    const int n = min(BLOCK, left), REC = VECS * DS + NUMBERS;
+    auto load = [&](const float* src, int c, float (&v)[4]) {                 // channels d .. d + 3 of the head's
+        const int d = (c * group + lane) * 4;
+        if (WIDE) {
+            const float4 f = d < p.dim ? *reinterpret_cast<const float4*>(src + at + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+        } else {
 #pragma unroll
-                for (int q = 0; q < VECS; ++q) v[q] = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int e = 0; e < 4; ++e) v[e] = d + e < p.dim ? src[at + d + e] : 0.f;
+        }
+    };
+    float w[BLOCK][CH][4], au[BLOCK][CH][4], k[BLOCK][CH][4];
+#pragma unroll
+    for (int b = 0; b < BLOCK; ++b) {
+        if (b >= n) break;
+        const float* row = p.proj + (size_t)(t + b) * p.ldp;
+        float u[CH][4], kk = 0.f;
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            load(row + p.k_col, c, k[b][c]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) kk = fmaf(k[b][c][e], k[b][c][e], kk);
+        }
+        const float inv = 1.0f / sqrtf(over_group(kk) + p.unit_eps);
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            float x[4], w0[4], a[4], a0[4];
+            load(p.x + (size_t)(t + b) * p.ldx, c, x);
+            load(p.w0, c, w0);
+            load(row + p.a_col, c, a);
+            load(p.a0, c, a0);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                w[b][c][e] = decay_exp(-p.decay_scale * sigmoid_f(x[e] + w0[e]));
+                u[c][e] = k[b][c][e] * inv;
+                au[b][c][e] = sigmoid_f(a[e] + a0[e]) * u[c][e];
             }
+        }
+        // from the token in front backwards: the products with its vectors, then its decay joins u
+        float numbers[NUMBERS] = {};
+        if (n == BLOCK) {
 #pragma unroll
-            for (int q = 0; q < VECS; ++q) *reinterpret_cast<float4*>(rec + q * DS + d) = v[q];
+            for (int j = b - 1; j >= 0; --j) {
+                float along_a = 0.f, along_k = 0.f;
+#pragma unroll
+                for (int c = 0; c < CH; ++c)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        along_a = fmaf(u[c][e], au[j][c][e], along_a);
+                        along_k = fmaf(u[c][e], k[j][c][e], along_k);
+                        u[c][e] *= w[j][c][e];
+                    }
+                numbers[j] = over_group(along_a);
+                numbers[4 + j] = over_group(along_k);
+            }
         }
-    } else {
-        for (int d = lane; d < DS; d += group) {
-            if (d < p.dim) put_channel(p, row, at, d, p.x[(size_t)t * p.ldx + at + d], inv, rec, DS);
-            else
-                for (int q = 0; q < VECS; ++q) rec[q * DS + d] = 0.f;
+        float* rec = p.records + ((size_t)h * p.tokens + t + b) * REC;
+        auto store = [&](int v, int c, const float (&f)[4], bool live) {
+            const int d = (c * group + lane) * 4;
+            if (d < DS)
+                *reinterpret_cast<float4*>(rec + v * DS + d) = live ? make_float4(f[0], f[1], f[2], f[3]) : make_float4(0.f, 0.f, 0.f, 0.f);
+        };
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            float r[4], v[4];
+            load(row + p.r_col, c, r);
+            load(row + p.v_col, c, v);
+            store(0, c, w[b][c], (c * group + lane) * 4 < p.dim);
+            store(1, c, u[c], true);
+            store(2, c, au[b][c], true);
+            store(3, c, k[b][c], true);
+            store(4, c, r, true);
+            store(5, c, v, true);
         }
+        if (lane < 2) *reinterpret_cast<float4*>(rec + VECS * DS + lane * 4) = lane ? make_float4(numbers[4], numbers[5], numbers[6], numbers[7])
+                                                                                       : make_float4(numbers[0], numbers[1], numbers[2], numbers[3]);
     }
 }
 
@@ -203,7 +253,7 @@ __global__ void __launch_bounds__(INLINE ? 512 : 256, 1) general_delta_kernel(co
     extern __shared__ __align__(128) float smem[];
     __shared__ __align__(8) uint64_t full[STAGES];
     __shared__ int abort_flag;
-    constexpr int DS = R * P, REC = VECS * DS, NSTAGES = INLINE ? 1 : STAGES;
+    constexpr int DS = R * P, REC = VECS * DS + NUMBERS, NSTAGES = INLINE ? 1 : STAGES;
     const int dim = p.dim, cols = p.cols, TILE = p.tile;
     float* s_o = smem + NSTAGES * TILE * REC;       // [2][TILE][cols]
     const int head = blockIdx.x, seq = blockIdx.y, j0 = blockIdx.z * cols;
@@ -370,28 +420,86 @@ __global__ void __launch_bounds__(INLINE ? 512 : 256, 1) general_delta_kernel(co
 #pragma unroll
             for (int c = 0; c < COLS; ++c) o[c] = sum_of(read[c][0]) + sum_of(read[c][1]);
         };
-        // The outputs of G = P / COLS tokens are P sums over P lanes: in every round a lane gives half of its sums away for the other half
-        // of a neighbour's, and ends with one of them.  Until then no shared memory is written, so that the loads of the group's tokens
-        // go out ahead of their steps.  (With a sum and a store after every token the loads of a token waited for the token before
-        // it: 445 cycles a token.)
-        constexpr int G = P / COLS;
         int t = 0;
-        for (; !INLINE && t + G <= n; t += G) {
-            float o[P];
+        for (; !INLINE && t + BLOCK <= n; t += BLOCK) {
+            const float* rec = base + t * REC + part * 4;
+            auto piece = [&](int b, int v, int i) { return *reinterpret_cast<const ulonglong2*>(rec + b * REC + v * DS + i * P * 4); };
+            float held[BLOCK][COLS], value[BLOCK][COLS];
 #pragma unroll
-            for (int i = 0; i < G; ++i) step(t + i, *reinterpret_cast<float (*)[COLS]>(&o[i * COLS]));
+            for (int b = 0; b < BLOCK; ++b) {
+                uint64_t sum[COLS][2] = {};
+#pragma unroll
+                for (int i = 0; i < R / 4; ++i) {
+                    const ulonglong2 u = piece(b, 1, i);
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) {
+                        sum[c][0] = fma2(s[c][2 * i], u.x, sum[c][0]);
+                        sum[c][1] = fma2(s[c][2 * i + 1], u.y, sum[c][1]);
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) {
+                    held[b][c] = sum_of(sum[c][0]) + sum_of(sum[c][1]);
+                    value[b][c] = base[(t + b) * REC + 5 * DS + j0 + jl + c];
+                }
+            }
+#pragma unroll
+            for (int x = 1; x < P; x <<= 1)
+#pragma unroll
+                for (int b = 0; b < BLOCK; ++b)
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) held[b][c] += __shfl_xor_sync(0xffffffffu, held[b][c], x);
+#pragma unroll
+            for (int b = 1; b < BLOCK; ++b) {
+                const float4 fa = *reinterpret_cast<const float4*>(base + (t + b) * REC + VECS * DS), fk = *reinterpret_cast<const float4*>(base + (t + b) * REC + VECS * DS + 4);
+                const float A[3] = {fa.x, fa.y, fa.z}, K[3] = {fk.x, fk.y, fk.z};
+#pragma unroll
+                for (int c = 0; c < COLS; ++c)
+#pragma unroll
+                    for (int j = 0; j < b; ++j) held[b][c] = fmaf(-A[j], held[j][c], fmaf(K[j], value[j][c], held[b][c]));
+            }
+            float o[BLOCK * COLS];
+#pragma unroll
+            for (int b = 0; b < BLOCK; ++b) {
+                uint64_t off2[COLS], value2[COLS], read[COLS][2] = {};
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) {
+                    off2[c] = pair_of(-held[b][c], -held[b][c]);
+                    value2[c] = pair_of(value[b][c], value[b][c]);
+                }
+#pragma unroll
+                for (int i = 0; i < R / 4; ++i) {
+                    const ulonglong2 w = piece(b, 0, i), a = piece(b, 2, i), k = piece(b, 3, i), q = piece(b, 4, i);
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) {
+                        s[c][2 * i] = fma2(w.x, s[c][2 * i], fma2(a.x, off2[c], mul2(k.x, value2[c])));
+                        s[c][2 * i + 1] = fma2(w.y, s[c][2 * i + 1], fma2(a.y, off2[c], mul2(k.y, value2[c])));
+                        read[c][0] = fma2(s[c][2 * i], q.x, read[c][0]);
+                        read[c][1] = fma2(s[c][2 * i + 1], q.y, read[c][1]);
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) o[b * COLS + c] = sum_of(read[c][0]) + sum_of(read[c][1]);
+            }
+            // the block's sums over the lanes: while a lane has several it gives half of them away for the other half of a neighbour's
             int which = 0;
 #pragma unroll
-            for (int x = 1, have = P / 2; x < P; x <<= 1, have >>= 1) {
-                const bool upper = part & x;
+            for (int x = 1, have = BLOCK * COLS; x < P; x <<= 1) {
+                if (have > 1) {
+                    have >>= 1;
+                    const bool upper = part & x;
 #pragma unroll
-                for (int i = 0; i < have; ++i) {
-                    const float give = upper ? o[i] : o[have + i], keep = upper ? o[have + i] : o[i];
-                    o[i] = keep + __shfl_xor_sync(0xffffffffu, give, x);
+                    for (int i = 0; i < have; ++i) {
+                        const float give = upper ? o[i] : o[have + i], keep = upper ? o[have + i] : o[i];
+                        o[i] = keep + __shfl_xor_sync(0xffffffffu, give, x);
+                    }
+                    which += upper ? have : 0;
+                } else {
+                    o[0] += __shfl_xor_sync(0xffffffffu, o[0], x);
                 }
-                which += upper ? have : 0;
             }
-            if (jl + which % COLS < width) out[(t + which / COLS) * cols + which % COLS] = o[0];
+            static_assert(BLOCK * COLS <= P, "a lane ends with one sum");
+            if (part < BLOCK * COLS && jl + which % COLS < width) out[(t + which / COLS) * cols + which % COLS] = o[0];
         }
         for (; t < n; ++t) {
             float o[COLS];
@@ -441,8 +549,7 @@ int power_of_two_lanes(int items) {                 // the least power of two th
 
 template <typename TO, int R, int P, int COLS, bool INLINE>
 int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num_seqs, bool float4_rows) {
-    constexpr int DS = R * P, REC = VECS * DS, per_warp = 32 / P * COLS;
-    static_assert(COLS <= P, "a lane ends with one column's sum");
+    constexpr int DS = R * P, REC = VECS * DS + NUMBERS, per_warp = 32 / P * COLS;
     const int most = (INLINE ? 512 : 256) / P * COLS / per_warp * per_warp;
     if (!p.o_raw) slices = 1;
     int cols = (p.dim + slices - 1) / slices;
@@ -461,10 +568,11 @@ int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num
     }
     const bool wide = float4_rows && p.dim % 4 == 0;
     if (!INLINE) {
-        p.lanes = power_of_two_lanes(wide ? DS / 4 : DS);
+        constexpr int CH = DS <= 128 ? 1 : 2;
+        p.lanes = DS / 4 / CH;
         const unsigned blocks = (unsigned)(((long long)p.tokens * p.heads * p.lanes + 255) / 256);
-        if (wide) general_delta_records_kernel<true><<<blocks, 256, 0, stream>>>(p, DS);
-        else general_delta_records_kernel<false><<<blocks, 256, 0, stream>>>(p, DS);
+        if (wide) general_delta_records_kernel<CH, true><<<blocks, 256, 0, stream>>>(p, DS);
+        else general_delta_records_kernel<CH, false><<<blocks, 256, 0, stream>>>(p, DS);
     }
     kernel<<<dim3(p.heads, num_seqs, slices), cols / COLS * P, smem, stream>>>(p);
     if (p.o_raw) {
@@ -483,8 +591,8 @@ int dispatch_general_delta(cudaStream_t stream, const DeltaParams& p, int slices
     if (p.dim <= 16) return launch_general_delta<TO, 4, 4, 1, INLINE>(stream, p, slices, num_seqs, wide);
     if (p.dim <= 32) return launch_general_delta<TO, 4, 8, 2, INLINE>(stream, p, slices, num_seqs, wide);
     if (p.dim <= 64) return launch_general_delta<TO, 8, 8, 2, INLINE>(stream, p, slices, num_seqs, wide);
-    if (p.dim <= 128) return launch_general_delta<TO, 8, 16, 4, INLINE>(stream, p, slices, num_seqs, wide);
-    return launch_general_delta<TO, 8, 32, 4, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 128) return launch_general_delta<TO, 8, 16, 2, INLINE>(stream, p, slices, num_seqs, wide);
+    return launch_general_delta<TO, 8, 32, 2, INLINE>(stream, p, slices, num_seqs, wide);
 }
 
 template <typename T>
@@ -497,7 +605,7 @@ __global__ void tanh_columns_kernel(const float* __restrict__ src, long long lds
 }  // namespace
 
 // float32 values of a record of a head of `dim` channels (scratch: heads * tokens of them)
-EG_API int eg_general_delta_record(int dim) { return VECS * (dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256); }
+EG_API int eg_general_delta_record(int dim) { return VECS * (dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256) + NUMBERS; }
 
 // up to how many tokens an entry may have, and how large the inner size may be, for eg_general_delta with x null
 EG_API int eg_general_delta_inline_takes(int entry_tokens, int rank) { return entry_tokens <= 8 && rank <= 512; }
@@ -510,8 +618,8 @@ EG_API int eg_general_delta_inline_takes(int entry_tokens, int rank) { return en
 // head's columns are dealt to that many blocks, and the outputs are normed by a kernel behind.  dim up to 256.
 EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ldp, int r_col, int k_col, int v_col, int g_col, int a_col, int inner_col,
                             const float* x, long long ldx, const void* w2, int ld2, int rank, const float* w0, const float* a0, const float* gain,
-                            float* records, float* state, long long slot_floats, long long state_offset, const int* seq_starts, const int* seq_slots,
-                            void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps,
+                            float* records, float* state, long long slot_floats, long long state_offset, const int* token_seq, const int* seq_starts,
+                            const int* seq_slots, void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps,
                             float eps, float decay_scale, int* status) {
     if (num_seqs <= 0 || tokens <= 0) return 0;
     if (heads <= 0 || dim <= 0 || dim > 256 || slices < 1 || (x && !records) || (!x && (!w2 || ld2 % 8 || (uintptr_t)w2 % 16))) return (int)cudaErrorInvalidValue;
@@ -539,6 +647,7 @@ EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ld
     p.state = state;
     p.slot_floats = slot_floats;
     p.state_offset = state_offset;
+    p.token_seq = token_seq;
     p.seq_starts = seq_starts;
     p.seq_slots = seq_slots;
     p.y = y;
