@@ -200,7 +200,7 @@ int eg_sigmoid_attention_tiles(cudaStream_t stream, const void* q, const void* k
 // attention_sigmoid.cu
 int eg_sigmoid_attention_split(cudaStream_t stream, const void* q, const void* k_cache, const void* v_cache, int row_stride, long long head_stride, const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* token_list, int num_tokens, const float* bias_table, int reach, const float* gate, long long ld_gate, void* out, long long ldo, float* partial, int* counters, int splits, int heads, int kv_heads, int dk, int dv, int page_size, long long page_stride, int num_pages, float scale, int* status);
 // general_delta.cu
-int eg_general_delta(cudaStream_t stream, const float* proj, long long ldp, int r_col, int k_col, int v_col, int g_col, int a_col, int inner_col, const float* x, long long ldx, const void* w2, int ld2, int rank, const float* w0, const float* a0, const float* gain, float* records, float* state, long long slot_floats, long long state_offset, const int* token_seq, const int* seq_starts, const int* seq_slots, void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps, float eps, float decay_scale, int* status);
+int eg_general_delta(cudaStream_t stream, const float* proj, long long ldp, int r_col, int k_col, int v_col, int g_col, int a_col, int inner_col, const float* x, long long ldx, const void* w2, int ld2, int rank, const float* w0, const float* a0, const float* gain, float* records, float* state, long long slot_floats, long long state_offset, const int* seq_starts, const int* seq_slots, void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps, float eps, float decay_scale, int* status);
 // general_delta.cu
 int eg_tanh_columns(cudaStream_t stream, const float* src, long long lds, void* dst, int dst_dtype, long long ldd, int rows, int cols, int padded);
 // lightning.cu

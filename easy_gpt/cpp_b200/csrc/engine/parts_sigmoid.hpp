@@ -382,7 +382,7 @@ public:
         float* o_raw = ctx.take<float>((size_t)T * n);
         launch_check(eg_general_delta(ctx.stream, (const float*)proj.p, proj.ld, 0, n, 2 * n, 3 * n, 4 * n, 5 * n, (const float*)x.p, x.ld, w2_.weight,
                                       w2_.in_features, rank_, w0_.as<float>(), a0_.as<float>(), norm_w_.as<float>(), records, (float*)cache.state, slot_floats(), 0,
-                                      ctx.token_seq, ctx.seq_starts, ctx.seq_slots, y.p, (int)dtype, y.ld, o_raw, plans::general_delta_slices(ctx.num_seqs, heads_, dim_), T,
+                                      ctx.seq_starts, ctx.seq_slots, y.p, (int)dtype, y.ld, o_raw, plans::general_delta_slices(ctx.num_seqs, heads_, dim_), T,
                                       ctx.num_seqs, heads_, dim_, unit_eps_, eps_, decay_scale_, ctx.status), "general_delta");
         const Rows o = out_(ctx, y, /*out_f32=*/true);
         Delta d;

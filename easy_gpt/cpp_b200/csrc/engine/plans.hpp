@@ -185,11 +185,11 @@ inline int delta_column_slices(int entries, int heads, int value_dim) {
     return (int)std::max<long long>(1, std::min<long long>(wanted, value_dim / 8));
 }
 
-// The same for the generalised delta rule: as many blocks as there are SMs, of at least one warp (8 columns; 4 or 2 of heads of
-// more than 64 or 128 rows).  Its warps read every token's vectors out of shared memory, whose rate is what the warps of an SM share.
+// The same for the generalised delta rule: as many blocks as there are SMs, of at least one warp (4 columns; 2 of heads of
+// more than 128 rows).  Its warps read every token's vectors out of shared memory, whose rate is what the warps of an SM share.
 inline int general_delta_slices(int entries, int heads, int dim) {
     const long long blocks = (long long)std::max(1, entries) * heads;
-    const int columns = dim <= 64 ? 8 : dim <= 128 ? 4 : 2;
+    const int columns = dim <= 128 ? 4 : 2;
     return (int)std::max<long long>(1, std::min<long long>((dim + columns - 1) / columns, sm_count() / blocks));
 }
 

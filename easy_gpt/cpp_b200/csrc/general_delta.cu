@@ -83,7 +83,7 @@ struct DeltaParams {
     float* records;             // [heads, tokens, VECS * DS + NUMBERS]
     float* state;
     long long slot_floats, state_offset;
-    const int *token_seq, *seq_starts, *seq_slots;
+    const int *seq_starts, *seq_slots;
     void* y;
     long long ldy;
     float* o_raw;               // [tokens, heads * dim], or null: the block holds whole heads
@@ -103,24 +103,16 @@ __device__ __forceinline__ void put_channel(const DeltaParams& p, const float* r
     rec[5 * DS + d] = row[p.v_col + at + d];
 }
 
-// `lanes` (a power of two up to 32) neighbouring lanes make the records of a block of tokens of a head: the group of the block's first
-// token does, the others have nothing to do.  A lane has CH runs of four channels; WIDE: by 16-byte loads.
-template <int CH, bool WIDE>
-__global__ void __launch_bounds__(256) general_delta_records_kernel(const DeltaParams p, int DS) {
-    const int group = p.lanes, lane = threadIdx.x % group;
-    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / group;
-    if (i >= (long long)p.tokens * p.heads) return;
-    // neighbouring groups take neighbouring heads of a token: the projection's rows are read in order
-    const int t = (int)(i / p.heads), h = (int)(i % p.heads), at = h * p.dim;
-    const int seq = p.token_seq[t], start = p.seq_starts[seq], left = p.seq_starts[seq + 1] - t;
-    if ((t - start) % BLOCK) return;
-    const unsigned mask = group == 32 ? 0xffffffffu : ((1u << group) - 1u) << (threadIdx.x % 32 / group * group);
+// The records of N tokens from token t on (a whole block, or one token of an incomplete one) of the head whose channels start at
+// `at`, by a group of lanes (`mask` in the warp), each with CH runs of four channels; WIDE: by 16-byte loads.
+template <int N, int CH, bool WIDE>
+__device__ __forceinline__ void make_records(const DeltaParams& p, int DS, int t, int h, int lane, int group, unsigned mask) {
+    const int at = h * p.dim, REC = VECS * DS + NUMBERS;
     auto over_group = [&](float v) {
         for (int o = group >> 1; o > 0; o >>= 1) v += __shfl_xor_sync(mask, v, o);
         return v;
     };
-    const int n = min(BLOCK, left), REC = VECS * DS + NUMBERS;
-    auto load = [&](const float* src, int c, float (&v)[4]) {                 // channels d .. d + 3 of the head's
+    auto load = [&](const float* src, int c, float (&v)[4]) {                 // the run's channels of the head
         const int d = (c * group + lane) * 4;
         if (WIDE) {
             const float4 f = d < p.dim ? *reinterpret_cast<const float4*>(src + at + d) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -130,72 +122,104 @@ __global__ void __launch_bounds__(256) general_delta_records_kernel(const DeltaP
             for (int e = 0; e < 4; ++e) v[e] = d + e < p.dim ? src[at + d + e] : 0.f;
         }
     };
-    float w[BLOCK][CH][4], au[BLOCK][CH][4], k[BLOCK][CH][4];
+    float w[N][CH][4], au[N][CH][4], k[N][CH][4], kk[N];
 #pragma unroll
-    for (int b = 0; b < BLOCK; ++b) {
-        if (b >= n) break;
+    for (int b = 0; b < N; ++b) {
         const float* row = p.proj + (size_t)(t + b) * p.ldp;
-        float u[CH][4], kk = 0.f;
+        kk[b] = 0.f;
 #pragma unroll
         for (int c = 0; c < CH; ++c) {
             load(row + p.k_col, c, k[b][c]);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) kk = fmaf(k[b][c][e], k[b][c][e], kk);
+            load(p.x + (size_t)(t + b) * p.ldx, c, w[b][c]);
+            load(row + p.a_col, c, au[b][c]);
         }
-        const float inv = 1.0f / sqrtf(over_group(kk) + p.unit_eps);
+    }
+    float w0[CH][4], a0[CH][4];
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        load(p.w0, c, w0[c]);
+        load(p.a0, c, a0[c]);
+    }
+#pragma unroll
+    for (int b = 0; b < N; ++b)
+#pragma unroll
+        for (int c = 0; c < CH; ++c)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) kk[b] = fmaf(k[b][c][e], k[b][c][e], kk[b]);
+#pragma unroll
+    for (int b = 0; b < N; ++b) kk[b] = over_group(kk[b]);
+#pragma unroll
+    for (int b = 0; b < N; ++b) {
+        const float* row = p.proj + (size_t)(t + b) * p.ldp;
+        float* rec = p.records + ((size_t)h * p.tokens + t + b) * REC;
+        auto store = [&](int v, int c, const float (&f)[4]) {
+            const int d = (c * group + lane) * 4;
+            if (d < DS) *reinterpret_cast<float4*>(rec + v * DS + d) = make_float4(f[0], f[1], f[2], f[3]);
+        };
+        const float inv = 1.0f / sqrtf(kk[b] + p.unit_eps);
+        float u[CH][4];
 #pragma unroll
         for (int c = 0; c < CH; ++c) {
-            float x[4], w0[4], a[4], a0[4];
-            load(p.x + (size_t)(t + b) * p.ldx, c, x);
-            load(p.w0, c, w0);
-            load(row + p.a_col, c, a);
-            load(p.a0, c, a0);
+            float f[4];
+            load(row + p.r_col, c, f);
+            store(4, c, f);
+            load(row + p.v_col, c, f);
+            store(5, c, f);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                w[b][c][e] = decay_exp(-p.decay_scale * sigmoid_f(x[e] + w0[e]));
+                w[b][c][e] = decay_exp(-p.decay_scale * sigmoid_f(w[b][c][e] + w0[c][e]));
                 u[c][e] = k[b][c][e] * inv;
-                au[b][c][e] = sigmoid_f(a[e] + a0[e]) * u[c][e];
+                au[b][c][e] = sigmoid_f(au[b][c][e] + a0[c][e]) * u[c][e];
             }
+            store(0, c, w[b][c]);
+            store(2, c, au[b][c]);
+            store(3, c, k[b][c]);
         }
         // from the token in front backwards: the products with its vectors, then its decay joins u
         float numbers[NUMBERS] = {};
-        if (n == BLOCK) {
 #pragma unroll
-            for (int j = b - 1; j >= 0; --j) {
-                float along_a = 0.f, along_k = 0.f;
+        for (int j = b - 1; j >= 0; --j) {
+            float along_a = 0.f, along_k = 0.f;
 #pragma unroll
-                for (int c = 0; c < CH; ++c)
+            for (int c = 0; c < CH; ++c)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        along_a = fmaf(u[c][e], au[j][c][e], along_a);
-                        along_k = fmaf(u[c][e], k[j][c][e], along_k);
-                        u[c][e] *= w[j][c][e];
-                    }
-                numbers[j] = over_group(along_a);
-                numbers[4 + j] = over_group(along_k);
-            }
+                for (int e = 0; e < 4; ++e) {
+                    along_a = fmaf(u[c][e], au[j][c][e], along_a);
+                    along_k = fmaf(u[c][e], k[j][c][e], along_k);
+                    u[c][e] *= w[j][c][e];
+                }
+            numbers[j] = over_group(along_a);
+            numbers[4 + j] = over_group(along_k);
         }
-        float* rec = p.records + ((size_t)h * p.tokens + t + b) * REC;
-        auto store = [&](int v, int c, const float (&f)[4], bool live) {
-            const int d = (c * group + lane) * 4;
-            if (d < DS)
-                *reinterpret_cast<float4*>(rec + v * DS + d) = live ? make_float4(f[0], f[1], f[2], f[3]) : make_float4(0.f, 0.f, 0.f, 0.f);
-        };
 #pragma unroll
-        for (int c = 0; c < CH; ++c) {
-            float r[4], v[4];
-            load(row + p.r_col, c, r);
-            load(row + p.v_col, c, v);
-            store(0, c, w[b][c], (c * group + lane) * 4 < p.dim);
-            store(1, c, u[c], true);
-            store(2, c, au[b][c], true);
-            store(3, c, k[b][c], true);
-            store(4, c, r, true);
-            store(5, c, v, true);
-        }
+        for (int c = 0; c < CH; ++c) store(1, c, u[c]);
         if (lane < 2) *reinterpret_cast<float4*>(rec + VECS * DS + lane * 4) = lane ? make_float4(numbers[4], numbers[5], numbers[6], numbers[7])
                                                                                        : make_float4(numbers[0], numbers[1], numbers[2], numbers[3]);
     }
+}
+
+// a group of p.lanes lanes (a power of two up to 32) per (block of tokens, head)
+template <int CH, bool WIDE>
+__global__ void __launch_bounds__(128) general_delta_records_kernel(const DeltaParams p, int DS, int num_seqs) {
+    const int group = p.lanes, lane = threadIdx.x % group;
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / group;
+    // neighbouring groups take neighbouring heads of a block: the projection's rows are read in order
+    int index = (int)(i / p.heads), t = -1, n = 0;
+    for (int s = 0; s < num_seqs; ++s) {
+        const int lo = p.seq_starts[s], count = p.seq_starts[s + 1] - lo, blocks = (count + BLOCK - 1) / BLOCK;
+        if (index < blocks) {
+            t = lo + index * BLOCK;
+            n = min(BLOCK, count - index * BLOCK);
+            break;
+        }
+        index -= blocks;
+    }
+    if (t < 0) return;
+    const int h = (int)(i % p.heads);
+    const unsigned mask = group == 32 ? 0xffffffffu : ((1u << group) - 1u) << (threadIdx.x % 32 / group * group);
+    if (n == BLOCK) make_records<BLOCK, CH, WIDE>(p, DS, t, h, lane, group, mask);
+    else
+        for (int b = 0; b < n; ++b) make_records<1, CH, WIDE>(p, DS, t + b, h, lane, group, mask);
 }
 
 // y = o / rms(o) * gain * sigmoid(g), a warp per (token, head)
@@ -570,9 +594,9 @@ int launch_general_delta(cudaStream_t stream, DeltaParams p, int slices, int num
     if (!INLINE) {
         constexpr int CH = DS <= 128 ? 1 : 2;
         p.lanes = DS / 4 / CH;
-        const unsigned blocks = (unsigned)(((long long)p.tokens * p.heads * p.lanes + 255) / 256);
-        if (wide) general_delta_records_kernel<CH, true><<<blocks, 256, 0, stream>>>(p, DS);
-        else general_delta_records_kernel<CH, false><<<blocks, 256, 0, stream>>>(p, DS);
+        const unsigned blocks = (unsigned)(((long long)(p.tokens / BLOCK + num_seqs) * p.heads * p.lanes + 127) / 128);
+        if (wide) general_delta_records_kernel<CH, true><<<blocks, 128, 0, stream>>>(p, DS, num_seqs);
+        else general_delta_records_kernel<CH, false><<<blocks, 128, 0, stream>>>(p, DS, num_seqs);
     }
     kernel<<<dim3(p.heads, num_seqs, slices), cols / COLS * P, smem, stream>>>(p);
     if (p.o_raw) {
@@ -590,7 +614,11 @@ template <typename TO, bool INLINE>
 int dispatch_general_delta(cudaStream_t stream, const DeltaParams& p, int slices, int num_seqs, bool wide) {
     if (p.dim <= 16) return launch_general_delta<TO, 4, 4, 1, INLINE>(stream, p, slices, num_seqs, wide);
     if (p.dim <= 32) return launch_general_delta<TO, 4, 8, 2, INLINE>(stream, p, slices, num_seqs, wide);
-    if (p.dim <= 64) return launch_general_delta<TO, 8, 8, 2, INLINE>(stream, p, slices, num_seqs, wide);
+    if (p.dim <= 64) {
+        // (prompts: half the rows a lane of what steps of short entries have, whose blocks hold whole heads)
+        if (INLINE) return launch_general_delta<TO, 8, 8, 2, INLINE>(stream, p, slices, num_seqs, wide);
+        return launch_general_delta<TO, 4, 16, 2, INLINE>(stream, p, slices, num_seqs, wide);
+    }
     if (p.dim <= 128) return launch_general_delta<TO, 8, 16, 2, INLINE>(stream, p, slices, num_seqs, wide);
     return launch_general_delta<TO, 8, 32, 2, INLINE>(stream, p, slices, num_seqs, wide);
 }
@@ -618,8 +646,8 @@ EG_API int eg_general_delta_inline_takes(int entry_tokens, int rank) { return en
 // head's columns are dealt to that many blocks, and the outputs are normed by a kernel behind.  dim up to 256.
 EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ldp, int r_col, int k_col, int v_col, int g_col, int a_col, int inner_col,
                             const float* x, long long ldx, const void* w2, int ld2, int rank, const float* w0, const float* a0, const float* gain,
-                            float* records, float* state, long long slot_floats, long long state_offset, const int* token_seq, const int* seq_starts,
-                            const int* seq_slots, void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps,
+                            float* records, float* state, long long slot_floats, long long state_offset, const int* seq_starts, const int* seq_slots,
+                            void* y, int y_dtype, long long ldy, float* o_raw, int slices, int tokens, int num_seqs, int heads, int dim, float unit_eps,
                             float eps, float decay_scale, int* status) {
     if (num_seqs <= 0 || tokens <= 0) return 0;
     if (heads <= 0 || dim <= 0 || dim > 256 || slices < 1 || (x && !records) || (!x && (!w2 || ld2 % 8 || (uintptr_t)w2 % 16))) return (int)cudaErrorInvalidValue;
@@ -647,7 +675,6 @@ EG_API int eg_general_delta(cudaStream_t stream, const float* proj, long long ld
     p.state = state;
     p.slot_floats = slot_floats;
     p.state_offset = state_offset;
-    p.token_seq = token_seq;
     p.seq_starts = seq_starts;
     p.seq_slots = seq_slots;
     p.y = y;
