@@ -3,6 +3,7 @@
 // state fades by a constant of the head; and the generalised delta rule with a decay and a removal rate per key channel.
 // Each takes its sizes, constants and tensor-name suffixes from its parameters and knows nothing of the model around it.
 #pragma once
+#include "../host/distance_bucket.hpp"
 #include "parts_delta.hpp"
 
 namespace easygpt::engine {
@@ -97,16 +98,6 @@ public:
         if (head_gate_) r.push_back(TensorRequest::matrix(prefix + ".g", heads_, hidden_));
         return r;
     }
-    // which row of a table of `rows` rows a distance reads
-    static int bucket(long long n, int rows, double most) {
-        const int half = rows / 2;
-        if (n < half) return (int)n;
-        if (half == 0 || most <= (double)half) return rows - 1;
-        const double grown = std::log((double)n / half) / std::log(most / half) * (rows - half);
-        // (a distance whose logarithm falls on a border mathematically, a power of the step, belongs to the upper row: the quotient of
-        // two rounded logarithms may fall a few 1e-16 short of it)
-        return (int)std::min<double>(rows - 1, half + std::floor(grown + 1e-11));
-    }
     void load(const HostTensors& file, DType dtype) override {
         std::vector<const char*> names = {".q", ".k", ".v"};
         if (head_gate_) names.push_back(".g");
@@ -134,14 +125,14 @@ public:
             const StoredTensor& t = need_tensor(file, prefix + ".rel");
             rel = host_floats(t);
             buckets = (int)t.shape[0];
-            while (bucket(reach_ - 1, buckets, bias_max_) < buckets - 1) ++reach_;
+            while (host::distance_bucket(reach_ - 1, buckets, bias_max_) < buckets - 1) ++reach_;
         }
         if (head_bias_) pb = host_floats(need_tensor(file, prefix + ".pb"));
         const float log2e = 1.4426950408889634f;
         std::vector<float> table((size_t)heads_ * reach_);
         for (int n = 0; n < reach_; ++n)
             for (int h = 0; h < heads_; ++h)
-                table[(size_t)h * reach_ + n] = (distance_bias_ ? rel[(size_t)bucket(n, buckets, bias_max_) * heads_ + h] : 0.f) + pb[h];
+                table[(size_t)h * reach_ + n] = (distance_bias_ ? rel[(size_t)host::distance_bucket(n, buckets, bias_max_) * heads_ + h] : 0.f) + pb[h];
         mma_ = dtype == DType::BF16 && eg_sigmoid_attention_mma_takes(dk_, dv_, reach_);
         if (mma_)
             for (float& v : table) v *= -log2e;               // the tensor-core kernels work on negated scores in base 2

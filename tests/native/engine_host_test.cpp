@@ -1,12 +1,14 @@
 // The native engine's host-only parts from C++ alone (no GPU, no CUDA headers): the JSON reader, the safetensors
 // reader with every malformed file refused, the one error that lists missing / unexpected / wrongly shaped tensors, the
 // typed Qwen2 configuration with what cannot run refused, the architecture registry's rule, and the run order's checks.
+#include <cmath>
 #include <cstdio>
 #include <cstring>
 #include <fstream>
 #include <functional>
 #include <iostream>
 
+#include "../host/distance_bucket.hpp"
 #include "architectures.hpp"
 #include "weights.hpp"
 
@@ -255,6 +257,74 @@ int main(int argc, char** argv) {
         bad = spec;
         bad.run_order[2].stream_add = 3;
         CHECK(throws<std::invalid_argument>([&] { bad.validate(); }, "names stream addition 3"));
+    }
+
+    // ---- a fifth listed design: norms in groups, waves of the position, two mixers side by side whose outputs are normed, a delta rule ----
+    {
+        const char* kFading = R"({"architecture": "Zodosun", "vocab": 83, "width": 60, "norm": {"eps": 2e-6, "groups": 3}, "logit_scale": 1.75,
+          "layers": [
+            {"type": "parallel", "mixer": {"left": {"heads": 6, "kv_heads": 2, "dim": 12, "vdim": 20, "scale": 0.4, "bias_max": 70, "q_temp": {"coef": 0.2, "every": 48}},
+                                           "right": {"heads": 2, "dim": 10, "vdim": 14, "decay": [0.75, 1]}},
+             "mlp": {"kind": "dense", "ff": 44}},
+            {"type": "general_delta", "mixer": {"heads": 5, "dim": 9}, "mlp": null},
+            {"type": "parallel", "mixer": {"left": {"heads": 1, "kv_heads": 1, "dim": 8, "vdim": 8, "scale": 1, "bias_max": 5.5},
+                                           "right": {"heads": 1, "dim": 4, "vdim": 6, "decay": [0.5]}}}]})";
+        const ModelSpec spec = ArchitectureRegistry::instance().build(json::parse(kFading));
+        CHECK(spec.architecture == "zodosun" && spec.layers.size() == 3 && spec.vocab_size == 83 && spec.hidden_size == 60 && spec.run_order.size() == 3);
+        for (int i = 0; i < 3; ++i) CHECK(spec.run_order[i].layer == i && spec.run_order[i].cache == i && spec.run_order[i].writes_cache);
+        CHECK(spec.embedding_position.present && spec.embedding_position.kind == "waves" && spec.embedding_position.params.integer("size") == 60 &&
+              spec.embedding_position.params.real("base") == 10000.0 && !spec.embedding.params.has("scale"));
+        CHECK(spec.lm_head.params.real("scale") == 1.75 && spec.final_norm.params.integer("groups") == 3 && spec.final_norm.prefix == "final.norm");
+        const SubLayerSpec& mix = spec.layers[0].sublayers[0];
+        CHECK(mix.norm.kind == "rmsnorm" && mix.norm.prefix == "l0.norm1" && mix.norm.params.integer("groups") == 3 && mix.norm.params.real("eps") == 2e-6 &&
+              mix.norm_placement == "pre" && !mix.output_norm.present && !spec.layers[0].parallel && !spec.layers[0].position.present);
+        CHECK(mix.part.kind == "side_by_side" && mix.part.prefix == "l0.mix" && mix.part.params.text("left_kind") == "sigmoid_attention" &&
+              mix.part.params.text("right_kind") == "lightning" && mix.part.params.real("norm_scale") == 0.5 && mix.part.params.real("norm_eps") == 2e-6 &&
+              mix.part.params.integer("hidden_size") == 60);
+        const Params left = mix.part.params.sub("left."), right = mix.part.params.sub("right.");
+        CHECK(left.integer("heads") == 6 && left.integer("kv_heads") == 2 && left.integer("dim") == 12 && left.integer("vdim") == 20 && left.real("scale") == 0.4 &&
+              left.real("bias_max") == 70 && left.real("temp_coef") == 0.2 && left.integer("temp_every") == 48 && left.real("norm_eps") == 2e-6 &&
+              left.integer("distance_bias") == 1 && left.integer("head_bias") == 1 && left.integer("head_gate") == 1 && left.integer("proj_bias") == 1);
+        CHECK(right.integer("heads") == 2 && right.integer("dim") == 10 && right.integer("vdim") == 14 && right.real("decay.0") == 0.75 && right.real("decay.1") == 1.0);
+        const SubLayerSpec& ff = spec.layers[0].sublayers[1];
+        CHECK(ff.part.kind == "swiglu" && ff.part.params.integer("intermediate_size") == 44 && ff.part.params.text("gate_name") == ".gate" && ff.part.prefix == "l0.mlp" &&
+              ff.norm.prefix == "l0.norm2");
+        const PartSpec& rule = spec.layers[1].sublayers[0].part;
+        CHECK(spec.layers[1].sublayers.size() == 1 && rule.kind == "general_delta" && rule.prefix == "l1.mix" && rule.params.integer("heads") == 5 &&
+              rule.params.integer("dim") == 9 && std::fabs(rule.params.real("decay_scale") - 0.6065306597126334) < 1e-15 && rule.params.real("unit_eps") == 1e-6 &&
+              !rule.params.has("rank"));
+        const Params plain = spec.layers[2].sublayers[0].part.params.sub("left.");
+        CHECK(spec.layers[2].sublayers.size() == 1 && !plain.has("temp_every") && plain.real("bias_max") == 5.5);
+        auto changed = [&](const std::string& from, const std::string& to) {
+            std::string text = kFading;
+            const size_t at = text.find(from);
+            CHECK(at != std::string::npos);
+            text.replace(at, from.size(), to);
+            return text;
+        };
+        const ModelSpec bare = ArchitectureRegistry::instance().build(json::parse(changed(R"(, "logit_scale": 1.75)", "")));
+        CHECK(!bare.lm_head.params.has("scale"));
+        const ModelSpec one_group = ArchitectureRegistry::instance().build(json::parse(changed(R"(, "groups": 3)", "")));
+        CHECK(one_group.final_norm.params.integer("groups") == 1);
+        for (const auto& wrong : {changed(R"("groups": 3)", R"("groups": 7)"), changed(R"("decay": [0.75, 1])", R"("decay": [0.75])"),
+                                  changed(R"("type": "general_delta")", R"("type": "delta")"), changed(R"("kv_heads": 2)", R"("kv_heads": 4)"),
+                                  changed(R"("every": 48)", R"("every": 0)"), changed(R"("kind": "dense")", R"("kind": "moe")"), changed(R"("bias_max": 70, )", "")}) {
+            bool refused = false;
+            try {
+                ArchitectureRegistry::instance().build(json::parse(wrong));
+            } catch (const std::exception&) {
+                refused = true;
+            }
+            CHECK(refused);
+        }
+        // the rows of a distance-bias table: one per distance, then growing ones, borders that are exact powers, odd and single rows
+        using easygpt::host::distance_bucket;
+        for (int n = 0; n < 8; ++n) CHECK(distance_bucket(n, 16, 128.0) == n);
+        const int borders[] = {8, 12, 16, 23, 32, 46, 64, 91};          // 8 * 2^(k / 2), the first whole distance of every further row
+        for (int k = 0; k < 8; ++k) CHECK(distance_bucket(borders[k], 16, 128.0) == 8 + k && distance_bucket(borders[k] - 1, 16, 128.0) == 7 + k);
+        CHECK(distance_bucket(128, 16, 128.0) == 15 && distance_bucket(1000000, 16, 128.0) == 15);
+        CHECK(distance_bucket(2, 7, 17.0) == 2 && distance_bucket(3, 7, 17.0) == 3 && distance_bucket(17, 7, 17.0) == 6 && distance_bucket(12, 7, 17.0) == 6);
+        CHECK(distance_bucket(0, 1, 9.0) == 0 && distance_bucket(50, 1, 9.0) == 0 && distance_bucket(0, 2, 9.0) == 0 && distance_bucket(1, 2, 9.0) == 1);
     }
 
     // ---- a fourth listed design: branches normed on their way back, masks of three kinds, two mixers side by side, shared tensors ----
