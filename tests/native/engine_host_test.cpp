@@ -291,7 +291,7 @@ int main(int argc, char** argv) {
               ff.norm.prefix == "l0.norm2");
         const PartSpec& rule = spec.layers[1].sublayers[0].part;
         CHECK(spec.layers[1].sublayers.size() == 1 && rule.kind == "general_delta" && rule.prefix == "l1.mix" && rule.params.integer("heads") == 5 &&
-              rule.params.integer("dim") == 9 && std::fabs(rule.params.real("decay_scale") - 0.6065306597126334) < 1e-15 && rule.params.real("unit_eps") == 1e-6 &&
+              rule.params.integer("dim") == 9 && rule.params.real("decay_scale") == std::exp(-0.5) && rule.params.real("unit_eps") == 1e-6 &&
               !rule.params.has("rank"));
         const Params plain = spec.layers[2].sublayers[0].part.params.sub("left.");
         CHECK(spec.layers[2].sublayers.size() == 1 && !plain.has("temp_every") && plain.real("bias_max") == 5.5);
