@@ -75,8 +75,9 @@ EG_API int eg_swiglu(cudaStream_t stream, int dtype, const void* gate_up, int ld
     return eg_launch_status();
 }
 
-// Two more activations between the products of a feed-forward, element by element in float32:
+// More activations between the products of a feed-forward, element by element in float32:
 //   eg_squared_relu   out[t, c] = max(x[t, c], 0)^2
+//   eg_gelu           out[t, c] = x Phi(x), Phi the normal distribution's integral: x / 2 (1 + erf(x / sqrt 2))
 //   eg_clamped_glu    on interleaved columns (gate_0, up_0, gate_1, up_1, ...): g = min(gate, limit), u = clamp(up, -limit, limit),
 //                     out[t, i] = g * sigmoid(1.702 g) * (u + 1)
 template <typename TI, typename TO>
@@ -127,4 +128,46 @@ EG_API int eg_clamped_glu_bias(cudaStream_t stream, const void* x, int x_dtype, 
 // x [tokens, 2 n] interleaved -> out [tokens, n]
 EG_API int eg_clamped_glu(cudaStream_t stream, const void* x, int x_dtype, long long ldx, void* out, int out_dtype, long long ldo, int tokens, int n, float limit) {
     return eg_clamped_glu_bias(stream, x, x_dtype, ldx, nullptr, out, out_dtype, ldo, tokens, n, limit);
+}
+
+namespace {
+template <typename TI, typename TO>
+__global__ void gelu_kernel(const TI* __restrict__ x, long long ldx, TO* __restrict__ out, long long ldo, int tokens, int n) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long long)tokens * n) return;
+    const int t = (int)(i / n), c = (int)(i % n);
+    out[(size_t)t * ldo + c] = from_f32<TO>(gelu_erf(to_f32<TI>(x[(size_t)t * ldx + c])));
+}
+
+// values[t, c] *= sigmoid(gate[t, c / span]), in place: span 1 has a gate per value, span v one for every run of v values (a head)
+template <typename T>
+__global__ void sigmoid_gate_kernel(T* __restrict__ values, long long ldv, const float* __restrict__ gate, long long ldg, int tokens, int n, int span) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long long)tokens * n) return;
+    const int t = (int)(i / n), c = (int)(i % n);
+    T* v = values + (size_t)t * ldv + c;
+    *v = from_f32<T>(to_f32<T>(*v) / (1.0f + expf(-gate[(size_t)t * ldg + c / span])));
+}
+}  // namespace
+
+EG_API int eg_gelu(cudaStream_t stream, const void* x, int x_dtype, long long ldx, void* out, int out_dtype, long long ldo, int tokens, int n) {
+    const long long total = (long long)tokens * n;
+    if (total <= 0) return 0;
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    if (x_dtype == EG_F32 && out_dtype == EG_F32) gelu_kernel<float, float><<<blocks, 256, 0, stream>>>((const float*)x, ldx, (float*)out, ldo, tokens, n);
+    else if (x_dtype == EG_F32) gelu_kernel<float, bf16><<<blocks, 256, 0, stream>>>((const float*)x, ldx, (bf16*)out, ldo, tokens, n);
+    else if (out_dtype == EG_F32) gelu_kernel<bf16, float><<<blocks, 256, 0, stream>>>((const bf16*)x, ldx, (float*)out, ldo, tokens, n);
+    else gelu_kernel<bf16, bf16><<<blocks, 256, 0, stream>>>((const bf16*)x, ldx, (bf16*)out, ldo, tokens, n);
+    return eg_launch_status();
+}
+
+// values [tokens, ldv] in dtype, n columns; gate float32 [tokens, ldg], n / span columns
+EG_API int eg_sigmoid_gate(cudaStream_t stream, int dtype, void* values, long long ldv, const float* gate, long long ldg, int tokens, int n, int span) {
+    const long long total = (long long)tokens * n;
+    if (total <= 0) return 0;
+    if (span < 1 || n % span) return (int)cudaErrorInvalidValue;
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    if (dtype == EG_BF16) sigmoid_gate_kernel<bf16><<<blocks, 256, 0, stream>>>((bf16*)values, ldv, gate, ldg, tokens, n, span);
+    else sigmoid_gate_kernel<float><<<blocks, 256, 0, stream>>>((float*)values, ldv, gate, ldg, tokens, n, span);
+    return eg_launch_status();
 }

@@ -13,8 +13,8 @@
 //                       (a learned logit per head that joins the denominator and has no value), float32
 //   eg_latent_expand    o [T, H, rank] -> [T, H * vdim] = Uv_h o
 //
-// The rotation turns neighbouring pairs (2i, 2i+1) of the first `rot_dims` values of the rotated part by the angle
-// position * inv_freq[i]; angles, sines and cosines are float32 (accurate sincosf).  Scores, weights, maxima and sums
+// The rotation turns pairs of the first `rot_dims` values of the rotated part, neighbours (2i, 2i+1) or with `rot_half` (i, i +
+// rot_dims/2), by the angle position * inv_freq[i]; angles, sines and cosines are float32 (accurate sincosf).  Scores, weights, maxima and sums
 // are float32; every sum's order depends on the token's own position only, never on the batch.
 #include "common.cuh"
 
@@ -26,7 +26,7 @@ __device__ __forceinline__ void store_any(void* p, int dtype, size_t i, float v)
 }
 
 // one block per token
-__global__ void latent_prepare_kernel(const float* __restrict__ down, long long ld, int q_rank, int rank, int rot, int rot_dims,
+__global__ void latent_prepare_kernel(const float* __restrict__ down, long long ld, int q_rank, int rank, int rot, int rot_dims, int rot_half,
                                       const float* __restrict__ gain_q, const float* __restrict__ gain_c, float eps, const float* __restrict__ inv_freq,
                                       const int* __restrict__ positions, const int* __restrict__ slot_map, void* __restrict__ cache, int cache_dtype,
                                       int page_size, long long page_stride, long long pool_slots, void* __restrict__ cq, int cq_dtype,
@@ -55,9 +55,10 @@ __global__ void latent_prepare_kernel(const float* __restrict__ down, long long 
     for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
         float sn, cs;
         sincosf(pos * inv_freq[i], &sn, &cs);
-        const float a = kr[2 * i], b = kr[2 * i + 1];
-        store_any(cache, cache_dtype, at + rank + 2 * i, a * cs - b * sn);
-        store_any(cache, cache_dtype, at + rank + 2 * i + 1, b * cs + a * sn);
+        const int d0 = rot_half ? i : 2 * i, d1 = rot_half ? i + rot_dims / 2 : 2 * i + 1;
+        const float a = kr[d0], b = kr[d1];
+        store_any(cache, cache_dtype, at + rank + d0, a * cs - b * sn);
+        store_any(cache, cache_dtype, at + rank + d1, b * cs + a * sn);
     }
     for (int j = rot_dims + threadIdx.x; j < rot; j += blockDim.x) store_any(cache, cache_dtype, at + rank + j, kr[j]);
 }
@@ -65,7 +66,7 @@ __global__ void latent_prepare_kernel(const float* __restrict__ down, long long 
 // one block per (token, head); Uk [heads * dim, rank] in TW
 template <typename TW>
 __global__ void latent_absorb_kernel(const float* __restrict__ q, long long ldq, const TW* __restrict__ Uk, const int* __restrict__ positions,
-                                     const float* __restrict__ inv_freq, int rot_dims, float scale, float* __restrict__ qa, int heads, int dim, int rot,
+                                     const float* __restrict__ inv_freq, int rot_dims, int rot_half, float scale, float* __restrict__ qa, int heads, int dim, int rot,
                                      int rank) {
     extern __shared__ float qs[];
     const int t = blockIdx.x, h = blockIdx.y;
@@ -84,9 +85,10 @@ __global__ void latent_absorb_kernel(const float* __restrict__ q, long long ldq,
     for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
         float sn, cs;
         sincosf(pos * inv_freq[i], &sn, &cs);
-        const float a = qr[2 * i], b = qr[2 * i + 1];
-        out[rank + 2 * i] = (a * cs - b * sn) * scale;
-        out[rank + 2 * i + 1] = (b * cs + a * sn) * scale;
+        const int d0 = rot_half ? i : 2 * i, d1 = rot_half ? i + rot_dims / 2 : 2 * i + 1;
+        const float a = qr[d0], b = qr[d1];
+        out[rank + d0] = (a * cs - b * sn) * scale;
+        out[rank + d1] = (b * cs + a * sn) * scale;
     }
     for (int j = rot_dims + threadIdx.x; j < rot; j += blockDim.x) out[rank + j] = qr[j] * scale;
 }
@@ -193,28 +195,28 @@ __global__ void latent_expand_kernel(const float* __restrict__ o, const TW* __re
 // down [T, ld] float32 holds per token (query latent [q_rank] | latent [rank] | rotated key part [rot]).  Writes the
 // unit-RMS query latent times gain_q to cq [T, q_rank] (cq_dtype), and unit-RMS latent times gain_c followed by the
 // rotated key part to the cache row of slot_map[t] (cache null: nothing is stored).  page_stride in elements.
-EG_API int eg_latent_prepare(cudaStream_t stream, const float* down, long long ld, int q_rank, int rank, int rot, int rot_dims, const float* gain_q,
+EG_API int eg_latent_prepare(cudaStream_t stream, const float* down, long long ld, int q_rank, int rank, int rot, int rot_dims, int rot_half, const float* gain_q,
                              const float* gain_c, float eps, const float* inv_freq, const int* positions, const int* slot_map, void* cache, int cache_dtype,
                              int page_size, long long page_stride, long long pool_slots, void* cq, int cq_dtype, int tokens, int* status) {
     if (tokens <= 0) return 0;
     if (rot_dims % 2 || rot_dims > rot || q_rank <= 0 || rank <= 0) return (int)cudaErrorInvalidValue;
-    latent_prepare_kernel<<<tokens, 128, 0, stream>>>(down, ld, q_rank, rank, rot, rot_dims, gain_q, gain_c, eps, inv_freq, positions, slot_map, cache,
+    latent_prepare_kernel<<<tokens, 128, 0, stream>>>(down, ld, q_rank, rank, rot, rot_dims, rot_half, gain_q, gain_c, eps, inv_freq, positions, slot_map, cache,
                                                      cache_dtype, page_size, page_stride, pool_slots, cq, cq_dtype, status);
     return eg_launch_status();
 }
 
 // qa [T, heads, rank + rot] float32 from q [T, ldq] float32 (head by head: dim plain values, rot rotated ones)
 EG_API int eg_latent_absorb(cudaStream_t stream, int w_dtype, const float* q, long long ldq, const void* Uk, const int* positions, const float* inv_freq,
-                            int rot_dims, float scale, float* qa, int tokens, int heads, int dim, int rot, int rank) {
+                            int rot_dims, int rot_half, float scale, float* qa, int tokens, int heads, int dim, int rot, int rank) {
     if (tokens <= 0) return 0;
     const size_t smem = (size_t)(dim + rot) * sizeof(float);
     if (smem > 48 * 1024 || rot_dims % 2 || rot_dims > rot) return (int)cudaErrorInvalidValue;
     dim3 grid(tokens, heads);
     const int threads = rank >= 256 ? 256 : 128;
     if (w_dtype == EG_BF16)
-        latent_absorb_kernel<bf16><<<grid, threads, smem, stream>>>(q, ldq, (const bf16*)Uk, positions, inv_freq, rot_dims, scale, qa, heads, dim, rot, rank);
+        latent_absorb_kernel<bf16><<<grid, threads, smem, stream>>>(q, ldq, (const bf16*)Uk, positions, inv_freq, rot_dims, rot_half, scale, qa, heads, dim, rot, rank);
     else
-        latent_absorb_kernel<float><<<grid, threads, smem, stream>>>(q, ldq, (const float*)Uk, positions, inv_freq, rot_dims, scale, qa, heads, dim, rot, rank);
+        latent_absorb_kernel<float><<<grid, threads, smem, stream>>>(q, ldq, (const float*)Uk, positions, inv_freq, rot_dims, rot_half, scale, qa, heads, dim, rot, rank);
     return eg_launch_status();
 }
 

@@ -274,7 +274,7 @@ __global__ void attention_latent_merge_kernel(const float* __restrict__ part_o, 
 
 // one thread per (token, head, pair): the rotated part of the query, scaled, into qa [T, heads, rank + rot]
 __global__ void latent_rotate_query_kernel(const bf16* __restrict__ q, long long ldq, const int* __restrict__ positions, const float* __restrict__ inv_freq,
-                                           int rot_dims, float scale, bf16* __restrict__ qa, int tokens, int heads, int dim, int rot, int rank) {
+                                           int rot_dims, int rot_half, float scale, bf16* __restrict__ qa, int tokens, int heads, int dim, int rot, int rank) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     const int half = (rot + 1) / 2;
     if (i >= (long long)tokens * heads * half) return;
@@ -282,12 +282,13 @@ __global__ void latent_rotate_query_kernel(const bf16* __restrict__ q, long long
     const bf16* src = q + (size_t)t * ldq + (size_t)h * (dim + rot) + dim;
     bf16* dst = qa + ((size_t)t * heads + h) * (rank + rot) + rank;
     const int d = 2 * pair;
-    if (d + 1 < rot_dims + 1 && d < rot_dims) {
+    if (d < rot_dims) {                             // as many pairs are turned as rot_dims has, neighbours or half of rot_dims apart
         float sn, cs;
         sincosf((float)positions[t] * inv_freq[pair], &sn, &cs);
-        const float a = __bfloat162float(src[d]), b = __bfloat162float(src[d + 1]);
-        dst[d] = __float2bfloat16_rn((a * cs - b * sn) * scale);
-        dst[d + 1] = __float2bfloat16_rn((b * cs + a * sn) * scale);
+        const int d0 = rot_half ? pair : d, d1 = rot_half ? pair + rot_dims / 2 : d + 1;
+        const float a = __bfloat162float(src[d0]), b = __bfloat162float(src[d1]);
+        dst[d0] = __float2bfloat16_rn((a * cs - b * sn) * scale);
+        dst[d1] = __float2bfloat16_rn((b * cs + a * sn) * scale);
     } else {
         dst[d] = __float2bfloat16_rn(__bfloat162float(src[d]) * scale);
         if (d + 1 < rot) dst[d + 1] = __float2bfloat16_rn(__bfloat162float(src[d + 1]) * scale);
@@ -327,12 +328,12 @@ EG_API int eg_attention_latent_mma(cudaStream_t stream, const void* qa, const vo
 }
 
 // the rotated, scaled part of the queries: qa[t, h, rank:] from q [T, ldq] (head by head: dim plain values, rot rotated ones)
-EG_API int eg_latent_rotate_query(cudaStream_t stream, const void* q, long long ldq, const int* positions, const float* inv_freq, int rot_dims, float scale,
-                                  void* qa, int tokens, int heads, int dim, int rot, int rank) {
+EG_API int eg_latent_rotate_query(cudaStream_t stream, const void* q, long long ldq, const int* positions, const float* inv_freq, int rot_dims, int rot_half,
+                                  float scale, void* qa, int tokens, int heads, int dim, int rot, int rank) {
     const long long n = (long long)tokens * heads * ((rot + 1) / 2);
     if (n <= 0) return 0;
     if (rot_dims % 2 || rot_dims > rot) return (int)cudaErrorInvalidValue;
-    latent_rotate_query_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>((const bf16*)q, ldq, positions, inv_freq, rot_dims, scale, (bf16*)qa, tokens, heads,
+    latent_rotate_query_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>((const bf16*)q, ldq, positions, inv_freq, rot_dims, rot_half, scale, (bf16*)qa, tokens, heads,
                                                                                dim, rot, rank);
     return eg_launch_status();
 }

@@ -20,7 +20,7 @@
 //
 // Attention.  The token at position p of its request sees key j <= p if
 //   (window <= 0 or p - j < window) and (chunk <= 0 or floor(j / chunk) == floor(p / chunk)), or if j < keep_first;
-//   score = (q . k) * scale, then with softcap > 0: softcap * tanh(score / softcap);
+//   score = (q . k) * scale, then with softcap > 0: softcap * tanh(score / softcap), then with slopes: minus slopes[row] * (p - j);
 //   weight_j = exp(s_j) / (sum_i exp(s_i) + (sinks ? exp(sinks[head row]) : 0)), the sink a term without a value;
 //   out = out_scale * sum_j weight_j v_j.
 // One warp per (token, query row), a running softmax over chunks of 32 keys that start at the first kept key and then at the
@@ -98,7 +98,7 @@ masked_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                         const int* __restrict__ block_table, int table_stride, const int* __restrict__ token_seq, const int* __restrict__ positions,
                         const int* __restrict__ token_list, TO* __restrict__ out, long long ldo, int heads, int kv_heads, int maps, int dk, int dv,
                         int page_size, long long page_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap,
-                        const float* __restrict__ sinks, float out_scale, int planes, int* status) {
+                        const float* __restrict__ sinks, const float* __restrict__ slopes, float out_scale, int planes, int* status) {
     extern __shared__ float q_shared[];              // WARPS * dk
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = token_list ? token_list[blockIdx.x] : blockIdx.x;
@@ -122,6 +122,7 @@ masked_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
 #pragma unroll
     for (int i = 0; i < MAX_PER_LANE; ++i) acc[i] = 0.0f;
     const float inv_cap = softcap > 0.f ? 1.0f / softcap : 0.f;
+    const float slope = slopes ? slopes[r] : 0.f;
     for (int part = 0; part < 2; ++part) {
         const int lo = part == 0 ? 0 : first, hi = part == 0 ? kept_end : pos + 1;      // keys lo .. hi - 1
         for (int base = lo; base < hi; base += 32) {
@@ -139,6 +140,7 @@ masked_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                 for (int d = 0; d < dk; ++d) dot = fmaf(qs[d], to_f32<T>(krow[d]), dot);
                 s = dot * scale;
                 if (softcap > 0.f) s = softcap * tanhf(s * inv_cap);
+                s = fmaf(slope, (float)(kpos - pos), s);
             }
             const float m_new = fmaxf(m, warp_max(s));
             if (m_new == -INFINITY) continue;
@@ -231,13 +233,13 @@ EG_API int eg_masked_attention_prepare(cudaStream_t stream, int dtype, const flo
 }
 
 // q [tokens, heads * maps, dk] in dtype; out [tokens, ldo] in out_dtype (the cache's dtype, or float32) with row r at column
-// r * dv.  token_list: the tokens to work on (num_tokens of them), or null for all.  sinks: float32 [heads * maps] or null.
+// r * dv.  token_list: the tokens to work on (num_tokens of them), or null for all.  sinks, slopes: float32 [heads * maps] or null.
 // Returns cudaErrorInvalidValue for sizes it does not take.
 EG_API int eg_masked_attention(cudaStream_t stream, int dtype, const void* q, const void* k_cache, const void* v_cache, int row_stride, long long head_stride,
                                const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* token_list, void* out,
                                int out_dtype, long long ldo, int num_tokens, int heads, int kv_heads, int maps, int dk, int dv, int page_size,
                                long long page_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks,
-                               float out_scale, int planes, int* status) {
+                               const float* slopes, float out_scale, int planes, int* status) {
     if (num_tokens <= 0) return 0;
     if (dv > 32 * MAX_PER_LANE || dv <= 0 || dk <= 0 || dk > 4096 || kv_heads <= 0 || heads % kv_heads || maps < 1 || keep_first < 0) return (int)cudaErrorInvalidValue;
     if (dtype == EG_F32 && out_dtype != EG_F32) return (int)cudaErrorInvalidValue;
@@ -246,7 +248,7 @@ EG_API int eg_masked_attention(cudaStream_t stream, int dtype, const void* q, co
 #define EG_MASKED(T, TO)                                                                                                                                     \
     masked_attention_kernel<T, TO><<<grid, WARPS * 32, smem, stream>>>((const T*)q, (const T*)k_cache, (const T*)v_cache, row_stride, head_stride, block_table, \
                                                                        table_stride, token_seq, positions, token_list, (TO*)out, ldo, heads, kv_heads, maps, dk, \
-                                                                       dv, page_size, page_stride, num_pages, window, chunk, keep_first, scale, softcap, sinks,  \
+                                                                       dv, page_size, page_stride, num_pages, window, chunk, keep_first, scale, softcap, sinks, slopes, \
                                                                        out_scale, planes, status)
     if (dtype == EG_BF16 && out_dtype == EG_BF16) EG_MASKED(bf16, bf16);
     else if (dtype == EG_BF16) EG_MASKED(bf16, float);

@@ -88,10 +88,12 @@ struct Params {
     // block of `chunk` positions only; keep_first: keys 0 .. keep_first - 1 stay visible whatever window and chunk say (their
     // key tiles are walked first); softcap c: the scaled score becomes c tanh(score / c); sinks: a logit per query row
     // (natural log) in place of sink2; maps m: query rows head * m + map read key head (head / group) * m + map (both planes
-    // hold num_kv_heads heads; num_heads counts rows); out_scale: a factor on the output; out_f32: float32 output [tokens, ldo].
+    // hold num_kv_heads heads; num_heads counts rows); slopes: per query row what a step of distance takes off the score;
+    // out_scale: a factor on the output; out_f32: float32 output [tokens, ldo].
     int chunk = 0, keep_first = 0, maps = 1;
     float softcap = 0.f, out_scale = 1.f;
     const float* sinks = nullptr;
+    const float* slopes = nullptr;
     float* out_f32 = nullptr;
 };
 
@@ -128,6 +130,7 @@ __global__ void __launch_bounds__(TPI * THREADS) attention_paged_kernel(const Pa
     const int split = blockIdx.z;
     const float scale_log2 = p.scale * 1.4426950408889634f;
     const float cap_pre = x_softcap > 0.f ? p.scale / x_softcap : 0.f, cap_post = x_softcap * 1.4426950408889634f;
+    const float* const x_slopes = MASKED ? p.slopes : nullptr;
     // the query row (and output row) of row r of this key head's group, and its sink (base 2)
     auto head_of = [&](int r) { return x_maps == 1 ? kvh * G + r : ((kvh / x_maps) * G + r) * x_maps + kvh % x_maps; };
     auto sink_of = [&](int r) { return x_sinks ? x_sinks[head_of(r)] * 1.4426950408889634f : p.sink2; };
@@ -289,6 +292,8 @@ __global__ void __launch_bounds__(TPI * THREADS) attention_paged_kernel(const Pa
             }
         }
         // scale, mask, running softmax
+        const float slope0 = x_slopes && g0 + gid < G ? x_slopes[head_of(g0 + gid)] * 1.4426950408889634f : 0.f;
+        const float slope1 = x_slopes && g0 + gid + 8 < G ? x_slopes[head_of(g0 + gid + 8)] * 1.4426950408889634f : 0.f;
         float tmax0 = -INFINITY, tmax1 = -INFINITY;
 #pragma unroll
         for (int j = 0; j < 2 * KB; ++j)
@@ -296,7 +301,9 @@ __global__ void __launch_bounds__(TPI * THREADS) attention_paged_kernel(const Pa
             for (int e = 0; e < 4; ++e) {
                 const int kpos = key_base + j * 8 + 2 * tig + (e & 1);
                 const bool ok = visible(kpos);
-                s[j][e] = ok ? (x_softcap > 0.f ? cap_post * tanh_by_exp(s[j][e] * cap_pre) : s[j][e] * scale_log2) : -INFINITY;
+                float x = x_softcap > 0.f ? cap_post * tanh_by_exp(s[j][e] * cap_pre) : s[j][e] * scale_log2;
+                if (MASKED) x = fmaf(e < 2 ? slope0 : slope1, (float)(kpos - pos), x);
+                s[j][e] = ok ? x : -INFINITY;
                 if (e < 2) tmax0 = fmaxf(tmax0, s[j][e]); else tmax1 = fmaxf(tmax1, s[j][e]);
             }
         tmax0 = fmaxf(tmax0, __shfl_xor_sync(0xffffffffu, tmax0, 1));
@@ -669,11 +676,12 @@ struct PrefillParams {
     // Further masks and score functions (all off by default).  chunk: a query sees keys of its own block of `chunk` positions
     // only; keep_first: keys 0 .. keep_first - 1 stay visible whatever window and chunk say; softcap c: the scaled score becomes
     // c tanh(score / c); sinks: a logit per query row in place of sink2; maps m: rows h = head * m + map read key head
-    // (head / group) * m + map (both planes hold num_kv_heads heads); out_scale: a factor on the output; out_f32: the
-    // output goes there as float32 [tokens, ldo] instead of to `out`.
+    // (head / group) * m + map (both planes hold num_kv_heads heads); slopes: per query row what a step of distance takes off the
+    // score; out_scale: a factor on the output; out_f32: the output goes there as float32 [tokens, ldo] instead of to `out`.
     int chunk = 0, keep_first = 0, maps = 1;
     float softcap = 0.f, out_scale = 1.f;
     const float* sinks = nullptr;
+    const float* slopes = nullptr;
     float* out_f32 = nullptr;
 };
 
@@ -700,8 +708,10 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 4 : 2) attention_prefill_k
     const int tile = item >> 1, half = item & 1;                 // a listed tile has up to 128 tokens: two CTAs
     const int h = blockIdx.y;
     const int kvh = (h / x_maps) / (p.num_heads / p.num_kv_heads) * x_maps + h % x_maps;
-    // with a soft cap the scores are scaled and capped as they come out of the product; else the scale rides in the exponent
-    const float scale_log2 = x_softcap > 0.f ? 1.4426950408889634f : p.scale * 1.4426950408889634f;
+    // with a soft cap or slopes the scores are finished as they come out of the product; else the scale rides in the exponent
+    const float* const x_slopes = MASKED ? p.slopes : nullptr;
+    const float scale_log2 = x_softcap > 0.f || x_slopes ? 1.4426950408889634f : p.scale * 1.4426950408889634f;
+    const float slope = x_slopes ? x_slopes[h] : 0.f;
     const float sink2 = x_sinks ? x_sinks[h] * 1.4426950408889634f : p.sink2;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int gid = lane >> 2, tig = lane & 3;
@@ -828,6 +838,13 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 4 : 2) attention_prefill_k
             for (int j = 0; j < 8; ++j)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) s[j][e] = x_softcap * tanh_by_exp(s[j][e] * pre);
+        }
+        if (x_slopes) {
+            const float mul = x_softcap > 0.f ? 1.f : p.scale;
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[j][e] = fmaf(s[j][e], mul, slope * (float)(key_base + j * 8 + 2 * tig + (e & 1) - (e < 2 ? qp0 : qp1)));
         }
         const bool limits = key_base + TILE_KEYS - 1 > warp_lo || warp * 16 + 15 >= count || key_base < first_of(warp_lo + 15);
         if (limits) {
@@ -961,6 +978,7 @@ static int attention_paged_any(cudaStream_t stream, const void* q, int ldq, cons
         p.softcap = extras->softcap;
         p.out_scale = extras->out_scale;
         p.sinks = extras->sinks;
+        p.slopes = extras->slopes;
         p.out_f32 = extras->out_f32;
     }
     if (extras) {
@@ -1045,13 +1063,13 @@ EG_API int eg_attention_prefill_sink(cudaStream_t stream, const void* q, int ldq
 
 // Prompt portions in tiles, with the further masks and score functions of PrefillParams: chunk (keys of the query's own block
 // of that many positions), keep_first (the first keys stay visible), softcap, sinks (float32 [num_heads], natural-log logits,
-// or null), maps (query row head * maps + map reads key head (head / group) * maps + map; num_heads and num_kv_heads count
+// or null), slopes (float32 [num_heads], natural units per step of distance, or null), maps (query row head * maps + map reads key head (head / group) * maps + map; num_heads and num_kv_heads count
 // rows and key heads, both planes hold num_kv_heads heads), out_scale; out_dtype EG_BF16, or EG_F32 for float32 rows.
 EG_API int eg_attention_prefill_masked(cudaStream_t stream, const void* q, int ldq, const void* k_cache, const void* v_cache, const int* block_table,
                                        int table_stride, const int* positions, const int* tiles, int num_tiles, void* out, int out_dtype, int ldo,
                                        int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride,
-                                       int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, float out_scale,
-                                       int* status) {
+                                       int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, const float* slopes,
+                                       float out_scale, int* status) {
     if (num_tiles <= 0) return 0;
     if (page_size % 16 || num_kv_heads <= 0 || num_heads % num_kv_heads || num_heads > 65535 || maps < 1 || num_kv_heads % maps || chunk < 0 || keep_first < 0 ||
         softcap < 0.f)
@@ -1064,6 +1082,7 @@ EG_API int eg_attention_prefill_masked(cudaStream_t stream, const void* q, int l
     p.maps = maps;
     p.softcap = softcap;
     p.sinks = sinks;
+    p.slopes = slopes;
     p.out_scale = out_scale;
     if (out_dtype == EG_F32) p.out_f32 = (float*)out;
     switch (head_dim) {
@@ -1075,13 +1094,13 @@ EG_API int eg_attention_prefill_masked(cudaStream_t stream, const void* q, int l
 }
 
 // Single tokens split over their keys, with the further masks and score functions of Params: chunk, keep_first, softcap, sinks
-// (float32 [num_heads], natural-log logits, or null), maps (num_heads and num_kv_heads count rows and key heads; both planes
-// hold num_kv_heads heads), out_scale; out_dtype EG_BF16, or EG_F32 for float32 rows (ldo a multiple of four then too).
+// (float32 [num_heads], natural-log logits, or null), slopes alike, maps (num_heads and num_kv_heads count rows and key heads; both
+// planes hold num_kv_heads heads), out_scale; out_dtype EG_BF16, or EG_F32 for float32 rows (ldo a multiple of four then too).
 EG_API int eg_attention_paged_masked(cudaStream_t stream, const void* q, int ldq, const void* k_cache, const void* v_cache, const int* block_table,
                                      int table_stride, const int* token_seq, const int* positions, const int* seq_context, void* out, int out_dtype, int ldo,
                                      float* partial_acc, float* partial_ml, int tokens, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size,
                                      long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale,
-                                     float softcap, const float* sinks, float out_scale, int splits, int* status, int* counters, int use_pdl,
+                                     float softcap, const float* sinks, const float* slopes, float out_scale, int splits, int* status, int* counters, int use_pdl,
                                      const int* token_list) {
     if (maps < 1 || num_kv_heads % maps || chunk < 0 || keep_first < 0 || softcap < 0.f || (out_dtype == EG_F32 && (ldo % 4 || (uintptr_t)out % 16)))
         return (int)cudaErrorInvalidValue;
@@ -1092,6 +1111,7 @@ EG_API int eg_attention_paged_masked(cudaStream_t stream, const void* q, int ldq
     extras.softcap = softcap;
     extras.out_scale = out_scale;
     extras.sinks = sinks;
+    extras.slopes = slopes;
     extras.out_f32 = out_dtype == EG_F32 ? (float*)out : nullptr;
     return attention_paged_any(stream, q, ldq, k_cache, v_cache, block_table, table_stride, token_seq, positions, seq_context, out, ldo, partial_acc,
                                partial_ml, tokens, num_heads, num_kv_heads, head_dim, page_size, page_stride, head_stride, num_pages, window, scale, splits,

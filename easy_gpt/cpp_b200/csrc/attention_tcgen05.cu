@@ -47,6 +47,9 @@
 // reference and no rescaling, and the parts of a cut key range simply add up (they carry reference 0 and sum 1).
 // weight = 1 / (1 + 2^x) with x = -log2(e) s: one exponent a score and one reciprocal for two scores (1 / a = b * 1 / (a b)).
 //
+// A fourth form (SLOPED) is the masked one with a distance's share in every score: slopes[row] * (p - j) is taken off, two more packed
+// multiply-adds a pair of scores as they come out of TMEM.
+//
 // Takes head sizes 64 and 128, pages of a multiple of 16 tokens, 16-byte aligned rows.  Anything else:
 // cudaErrorInvalidValue, and the caller uses the warp-level kernel.
 #define EG_NEEDS_TENSOR_MAPS
@@ -244,6 +247,7 @@ struct Params {
     int chunk = 0, keep_first = 0, maps = 1;
     float out_scale = 1.f;
     const float* sinks = nullptr;
+    const float* slopes = nullptr;          // SLOPED: per query row what a step of distance takes off the score
     float* out_f32 = nullptr;
     // SIGMOID: -log2(e) times the bias of every head by distance [num_heads, reach], the gates' logits [tokens, ld_gate] (head h at
     // column h, or null); `scale` is then -log2(e) times the scores' factor
@@ -252,7 +256,7 @@ struct Params {
     const float* gate = nullptr;
     long long ld_gate = 0;
 };
-enum Form { PLAIN = 0, MASKED_FORM = 1, SIGMOID = 2 };
+enum Form { PLAIN = 0, MASKED_FORM = 1, SIGMOID = 2, SLOPED = 3 };
 constexpr int BIAS_ENTRIES = 2048;                                // of a head's table, in shared memory
 
 // two weights 1 / (1 + 2^x0), 1 / (1 + 2^x1) with one reciprocal (x is kept below 60, where the weight is 1e-18, so that the product
@@ -310,7 +314,7 @@ __global__ void __launch_bounds__((Shape<HD, WGS>::THREADS), (Shape<HD, WGS>::CT
 attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                  const __grid_constant__ CUtensorMap map_v, const Params p) {
     using S = Shape<HD, WGS>;
-    constexpr bool MASKED = FORM == MASKED_FORM;
+    constexpr bool MASKED = FORM == MASKED_FORM || FORM == SLOPED;
     const int x_keep = MASKED ? p.keep_first : 0, x_maps = MASKED ? p.maps : 1;
     const float x_out_scale = MASKED ? p.out_scale : 1.f;
     float* const x_out_f32 = MASKED ? p.out_f32 : nullptr;
@@ -537,7 +541,9 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
             const int warp_lo = pos_lo + quad * 32, warp_hi = pos_lo + min(count - 1, quad * 32 + 31);
             const int warp_first = first_visible<MASKED>(p, warp_lo), row_first = first_visible<MASKED>(p, qpos);
             const bool warp_has_rows = quad * 32 < count;
-            const float scale_log2 = p.scale * 1.4426950408889634f;
+            // SLOPED: the scores are brought to base-2 units as they come out of TMEM
+            const float scale_log2 = FORM == SLOPED ? 1.f : p.scale * 1.4426950408889634f;
+            const float slope2 = FORM == SLOPED ? p.slopes[h] * 1.4426950408889634f : 0.f;
             const uint32_t lane_base = tmem_base + ((uint32_t)(quad * 32) << 16);
             const uint32_t o_lane = lane_base + (uint32_t)(S::O_COL + g * HD);
 
@@ -576,6 +582,13 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                         }
                     }
                     STAMP(2)
+                    if constexpr (FORM == SLOPED) {
+                        const float mul = p.scale * 1.4426950408889634f, at = slope2 * (float)(key_base - qpos);
+                        const uint64_t mul2 = pair_of(mul, mul), at2 = pair_of(at, at), slopes2 = pair_of(slope2, slope2);
+#pragma unroll
+                        for (int e = 0; e < 64; e += 2)
+                            split_pair(fma_pair(pair_of(s[e], s[e + 1]), mul2, fma_pair(slopes2, pair_of((float)e, (float)(e + 1)), at2)), s[e], s[e + 1]);
+                    }
                     if constexpr (FORM != SIGMOID) {
                     // only a tile that crosses the diagonal, the window's far edge or the end of the portion needs limits
                     // (also a tile with kept first keys, and one in which a chunk of some row of the warp begins)
@@ -821,7 +834,7 @@ constexpr int MERGE_MAX_PARTS = 8;
 template <int HD, int FORM>
 __global__ void __launch_bounds__(256)
 attention_merge_parts_kernel(const Params p) {
-    constexpr bool MASKED = FORM == MASKED_FORM;
+    constexpr bool MASKED = FORM == MASKED_FORM || FORM == SLOPED;
     const float x_out_scale = MASKED ? p.out_scale : 1.f;
     float* const x_out_f32 = MASKED ? p.out_f32 : nullptr;
     asm volatile("griddepcontrol.wait;\n" ::: "memory");
@@ -971,6 +984,7 @@ static int attention_prefill_tcgen05_any(cudaStream_t stream, const void* q, lon
         p.maps = extras->maps;
         p.out_scale = extras->out_scale;
         p.sinks = extras->sinks;
+        p.slopes = extras->slopes;
         p.out_f32 = extras->out_f32;
         p.bias_table = extras->bias_table;
         p.reach = extras->reach;
@@ -997,10 +1011,12 @@ static int attention_prefill_tcgen05_any(cudaStream_t stream, const void* q, lon
     static const int asked = getenv("EASY_GPT_PREFILL_GROUPS") ? atoi(getenv("EASY_GPT_PREFILL_GROUPS")) : 0;
     const int groups = asked == 1 || asked == 2 ? asked : eg_attention_prefill_groups(head_dim);
     int code;
-    const int form = !extras ? PLAIN : extras->bias_table ? SIGMOID : MASKED_FORM;
+    const int form = !extras ? PLAIN : extras->bias_table ? SIGMOID : extras->slopes ? SLOPED : MASKED_FORM;
 #define EG_FORM(WGS, F) (head_dim == 64 ? launch<64, WGS, F>(stream, map_q, map_k, map_v, p, sm_count) : launch<128, WGS, F>(stream, map_q, map_k, map_v, p, sm_count))
-    if (groups == 1) code = form == SIGMOID ? EG_FORM(1, SIGMOID) : form == MASKED_FORM ? EG_FORM(1, MASKED_FORM) : EG_FORM(1, PLAIN);
-    else code = form == SIGMOID ? EG_FORM(2, SIGMOID) : form == MASKED_FORM ? EG_FORM(2, MASKED_FORM) : EG_FORM(2, PLAIN);
+    if (groups == 1)
+        code = form == SIGMOID ? EG_FORM(1, SIGMOID) : form == SLOPED ? EG_FORM(1, SLOPED) : form == MASKED_FORM ? EG_FORM(1, MASKED_FORM) : EG_FORM(1, PLAIN);
+    else
+        code = form == SIGMOID ? EG_FORM(2, SIGMOID) : form == SLOPED ? EG_FORM(2, SLOPED) : form == MASKED_FORM ? EG_FORM(2, MASKED_FORM) : EG_FORM(2, PLAIN);
 #undef EG_FORM
     if (code || max_parts == 1) return code;
     // the parts are added up behind the main kernel (launched early: it waits for it by itself)
@@ -1017,7 +1033,7 @@ static int attention_prefill_tcgen05_any(cudaStream_t stream, const void* q, lon
     return (int)(head_dim == 64 ? cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<64, F>, p) \
                                 : cudaLaunchKernelEx(&cfg, attention_merge_parts_kernel<128, F>, p))
     if (form == SIGMOID) EG_MERGE(SIGMOID);
-    if (form == MASKED_FORM) EG_MERGE(MASKED_FORM);
+    if (form == MASKED_FORM || form == SLOPED) EG_MERGE(MASKED_FORM);
     EG_MERGE(PLAIN);
 #undef EG_MERGE
 }
@@ -1045,14 +1061,14 @@ EG_API int eg_attention_prefill_tcgen05_sink(cudaStream_t stream, const void* q,
                                          max_parts, part_tiles, partial_o, partial_ml, queue, sink_logit * 1.4426950408889634f);
 }
 
-// The same with the further masks of Params: chunk, keep_first, sinks (float32 [num_heads], natural-log logits, or null),
-// maps (num_heads and num_kv_heads count rows and key heads; both planes hold num_kv_heads
+// The same with the further masks of Params: chunk, keep_first, sinks (float32 [num_heads], natural-log logits, or null), slopes
+// (float32 [num_heads], natural units per step of distance, or null), maps (num_heads and num_kv_heads count rows and key heads; both planes hold num_kv_heads
 // heads), out_scale; out_dtype EG_BF16, or EG_F32 for float32 rows.
 EG_API int eg_attention_prefill_tcgen05_masked(cudaStream_t stream, const void* q, long long ldq, int total_tokens, const void* k_cache, const void* v_cache,
                                                const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, void* out,
                                                int out_dtype, long long ldo, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size,
                                                long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale,
-                                               const float* sinks, float out_scale, int* status, int max_parts, int part_tiles, float* partial_o,
+                                               const float* sinks, const float* slopes, float out_scale, int* status, int max_parts, int part_tiles, float* partial_o,
                                                float* partial_ml, int* queue) {
     if (maps < 1 || num_kv_heads % maps || chunk < 0 || keep_first < 0) return (int)cudaErrorInvalidValue;
     Params extras{};
@@ -1061,6 +1077,7 @@ EG_API int eg_attention_prefill_tcgen05_masked(cudaStream_t stream, const void* 
     extras.maps = maps;
     extras.out_scale = out_scale;
     extras.sinks = sinks;
+    extras.slopes = slopes;
     extras.out_f32 = out_dtype == EG_F32 ? (float*)out : nullptr;
     return attention_prefill_tcgen05_any(stream, q, ldq, total_tokens, k_cache, v_cache, block_table, table_stride, positions, tiles, num_tiles, out, ldo,
                                          num_heads, num_kv_heads, head_dim, page_size, page_stride, head_stride, num_pages, window, scale, status, nullptr,

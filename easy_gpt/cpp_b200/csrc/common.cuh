@@ -41,6 +41,9 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// z times the normal distribution's integral up to z
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+
 // Sum over a block of up to 1024 threads; every thread gets the result.  The
 // order of the additions depends only on blockDim, never on the data or on what
 // else is in the batch.  `scratch` holds 32 floats of shared memory.

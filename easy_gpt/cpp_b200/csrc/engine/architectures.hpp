@@ -832,6 +832,135 @@ inline ModelSpec zodosun_spec(const json::Value& config) {
     return spec;
 }
 
+// ---- Mipurax ---------------------------------------------------------------------------------------------------------------
+// A decoder whose config.json lists its layers one by one.  The stream starts as the norm of the embedding; a layer is
+// x = x + mixer(n1(x)), x = x + ff(n2(x)) (or the mixer alone), all norms RMS norms whose tensors hold the gain minus one; the output is
+// the model's norm and the embedding table.  The mixer is one of three: "latent_attention" and "latent_attention_2" (attention through
+// a cached latent with a gate on its output: neighbouring pairs turned and a gate per value, or halves turned, a sink per head and a
+// gate per head) and "attention" (grouped heads without rotation, a distance bias with a slope per head, keys of the query's own block
+// of mask.size positions).  An "attention" with "kv_from": j has queries of its own and reads the keys and values of layer j.  "mlp" is
+// null, a dense feed-forward with the exact gelu, or routed experts of that form (sigmoid scores, choice within the best groups,
+// weights that sum to one) beside a shared one.  Every size and constant is a key of config.json; tensor names are
+// "l<i>.<part>.<tensor>".
+inline ModelSpec mipurax_spec(const json::Value& config) {
+    using C = GufanexConfig;        // the typed readers (a key's path goes into the refusal)
+    if (!config.is_object()) throw ConfigError("config.json is not a JSON object");
+    ModelSpec spec;
+    spec.architecture = "mipurax";
+    auto positive = [&](const json::Value& m, const char* key, const std::string& w) {
+        const long long v = C::integer(m, key, w);
+        if (v <= 0) throw ConfigError(w + key + " must be > 0");
+        return v;
+    };
+    const long long width = positive(config, "width", ""), vocab = positive(config, "vocab", "");
+    const double eps = C::number(C::need(config, "norm", ""), "eps", "norm.");
+    if (eps <= 0.0) throw ConfigError("norm.eps must be > 0");
+    spec.vocab_size = vocab;
+    spec.hidden_size = width;
+    spec.max_positions = C::integer_or(config, "max_positions", 1LL << 30, "");     // the design sets no limit; positions are 32-bit
+    auto norm = [&](const std::string& name) {
+        return PartSpec{"rmsnorm", Params{{"size", width}, {"eps", eps}, {"weight_name", ""}, {"offset", 1.0}}, name, true};
+    };
+    const json::Value& layers = C::need(config, "layers", "");
+    if (!layers.is_array() || layers.array.empty()) throw ConfigError("layers must be a list with at least one layer");
+    const long long count = (long long)layers.array.size();
+    // whose keys an attention layer reads, its chunk (0: all earlier keys), and how far back any layer looks into a layer's cache (-1: all)
+    std::vector<long long> source(count), chunk(count, 0), back(count, 0);
+    for (long long i = 0; i < count; ++i) {
+        const std::string where = "layers[" + std::to_string(i) + "].", w = where + "mixer.";
+        const json::Value &type = C::need(layers.array[i], "type", where), &m = C::need(layers.array[i], "mixer", where);
+        if (!type.is_string()) throw ConfigError(where + "type must be a string");
+        source[i] = i;
+        if (type.string != "attention") continue;
+        if (C::present(m, "mask")) chunk[i] = positive(*m.find("mask"), "size", w + "mask.");
+        if (C::present(m, "kv_from")) {
+            const long long j = C::integer(m, "kv_from", w);
+            if (j < 0 || j >= i || layers.array[j].find("type")->string != "attention" || source[j] != j)
+                throw ConfigError(w + "kv_from must name an attention layer in front of it that has keys of its own");
+            for (const char* key : {"heads", "kv_heads", "dim", "vdim"})
+                if (C::integer(m, key, w) != C::integer(*layers.array[j].find("mixer"), key, w))
+                    throw ConfigError(w + key + " differs from that of the layer whose keys it reads");
+            source[i] = j;
+        }
+        long long& reach = back[source[i]];
+        if (reach >= 0) reach = chunk[i] == 0 ? -1 : std::max(reach, chunk[i]);
+    }
+    for (long long i = 0; i < count; ++i) {
+        const json::Value& l = layers.array[i];
+        const std::string where = "layers[" + std::to_string(i) + "].", prefix = "l" + std::to_string(i), w = where + "mixer.";
+        const json::Value& m = *l.find("mixer");
+        const std::string& type = l.find("type")->string;
+        const bool second = type == "latent_attention_2";
+        PartSpec mixer;
+        if (type == "latent_attention" || second) {
+            Params a{{"hidden_size", width}, {"heads", positive(m, "heads", w)}, {"dim", positive(m, "dim", w)}, {"rot_dim", C::integer(m, "rot_dim", w)},
+                     {"vdim", positive(m, "vdim", w)}, {"kv_rank", positive(m, "kv_rank", w)}, {"q_rank", positive(m, "q_rank", w)},
+                     {"scale", C::number(m, "scale", w)}, {"eps", eps}, {"sink", second}, {"rot_layout", second ? "half" : "interleaved"},
+                     {"gate", second ? "heads" : "values"}};
+            const long long rot_dim = a.integer("rot_dim");
+            if (rot_dim < 0) throw ConfigError(w + "rot_dim must not be negative");
+            a.set("rot_dims", 0LL);
+            a.set("rot_base", 1.0);
+            if (rot_dim > 0) {
+                const json::Value& rot = C::need(m, "rot", w);
+                const long long dims = C::integer_or(rot, "dims", rot_dim, w + "rot.");
+                if (dims < 0 || dims % 2 || dims > rot_dim) throw ConfigError(w + "rot.dims must be even and within rot_dim");
+                a.set("rot_dims", dims);
+                a.set("rot_base", C::number(rot, "base", w + "rot."));
+            }
+            mixer = PartSpec{"latent_attention", a, prefix + ".mix", true};
+        } else if (type == "attention") {
+            Params a{{"hidden_size", width}, {"heads", positive(m, "heads", w)}, {"kv_heads", positive(m, "kv_heads", w)}, {"dim", positive(m, "dim", w)},
+                     {"vdim", positive(m, "vdim", w)}, {"scale", C::number(m, "scale", w)}, {"slopes", 1}, {"own_keys", source[i] == i ? 1 : 0},
+                     {"cached_back", back[source[i]]}};
+            if (a.integer("heads") % a.integer("kv_heads")) throw ConfigError(w + "heads must be a multiple of kv_heads");
+            if (chunk[i] > 0) a.set("chunk", chunk[i]);
+            mixer = PartSpec{"masked_attention", a, prefix + ".mix", true};
+        } else {
+            throw ConfigError(where + "type '" + type + "' is no mixer of this design (latent_attention, latent_attention_2, attention)");
+        }
+        LayerSpec layer;
+        layer.sublayers.push_back({"mixer", mixer, norm(prefix + ".norm1"), "pre", PartSpec::none()});
+        if (C::present(l, "mlp")) {
+            const json::Value& mlp = *l.find("mlp");
+            const std::string wm = where + "mlp.";
+            const json::Value& kind = C::need(mlp, "kind", wm);
+            if (!kind.is_string()) throw ConfigError(wm + "kind must be a string");
+            PartSpec ff;
+            if (kind.string == "dense") {
+                ff = PartSpec{"gelu", Params{{"hidden_size", width}, {"ff", positive(mlp, "ff", wm)}}, prefix + ".mlp", true};
+            } else if (kind.string == "moe") {
+                const json::Value& router = C::need(mlp, "router", wm);
+                const std::string wr = wm + "router.";
+                Params e{{"hidden_size", width}, {"experts", positive(router, "experts", wr)}, {"top", positive(router, "top", wr)},
+                         {"ff", positive(C::need(mlp, "expert", wm), "ff", wm + "expert.")}, {"scoring", "sigmoid"}, {"correction", 0}, {"activation", "gelu"},
+                         {"normalize", 1}, {"shared_gated", 0}};
+                if (C::present(router, "groups")) {
+                    const json::Value& groups = *router.find("groups");
+                    e.set("groups", positive(groups, "count", wr + "groups."));
+                    e.set("keep_groups", positive(groups, "keep", wr + "groups."));
+                    if (e.integer("experts") % e.integer("groups") || e.integer("keep_groups") > e.integer("groups"))
+                        throw ConfigError(wr + "groups.count must divide experts, and groups.keep must not exceed it");
+                }
+                if (e.integer("top") > e.integer("experts") / e.integer("groups", 1) * e.integer("keep_groups", 1))
+                    throw ConfigError(wr + "top exceeds what can be chosen");
+                if (C::present(mlp, "shared")) e.set("shared_ff", positive(*mlp.find("shared"), "ff", wm + "shared."));
+                ff = PartSpec{"routed_experts", e, prefix + ".mlp", true};
+            } else {
+                throw ConfigError(wm + "kind '" + kind.string + "' is no feed-forward of this design (dense, moe)");
+            }
+            layer.sublayers.push_back({"feed_forward", ff, norm(prefix + ".norm2"), "pre", PartSpec::none()});
+        }
+        spec.layers.push_back(std::move(layer));
+        spec.run_order.push_back(RunEntry{(int)i, (int)source[i], source[i] == i});
+    }
+    spec.embedding = PartSpec{"embedding", Params{{"vocab_size", vocab}, {"hidden_size", width}, {"weight_name", ""}, {"norm_name", ".norm"}, {"norm_eps", eps},
+                                                  {"norm_offset", 1.0}}, "embed", true};
+    spec.final_norm = norm("final.norm");
+    spec.lm_head = PartSpec{"lm_head", Params{{"vocab_size", vocab}, {"hidden_size", width}, {"tied_to", "embed"}}, "head", true};
+    return spec;
+}
+
 inline void register_builtin_architectures() {
     ArchitectureRegistry& r = ArchitectureRegistry::instance();
     for (auto& e : r.entries)
@@ -842,6 +971,7 @@ inline void register_builtin_architectures() {
     r.add("masezen", masezen_spec);
     r.add("mozalix", mozalix_spec);
     r.add("zodosun", zodosun_spec);
+    r.add("mipurax", mipurax_spec);
 }
 
 }  // namespace easygpt::engine

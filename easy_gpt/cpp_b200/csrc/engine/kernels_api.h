@@ -62,15 +62,15 @@ int eg_step_sizes(cudaStream_t stream, const float* low, long long ldl, const fl
 // selective_scan.cu
 int eg_selective_scan(cudaStream_t stream, int dtype, const void* u, long long ldu, const float* dt, const float* dt_bias, const float* low, long long ldl, int b_col, int c_col, const float* A, const float* D, const void* z, long long ldz, float* state, long long slot_floats, long long state_offset, const int* seq_starts, const int* seq_slots, void* y, long long ldy, int num_seqs, int channels, int states, int states_per_lane);
 // attention_latent.cu
-int eg_latent_prepare(cudaStream_t stream, const float* down, long long ld, int q_rank, int rank, int rot, int rot_dims, const float* gain_q, const float* gain_c, float eps, const float* inv_freq, const int* positions, const int* slot_map, void* cache, int cache_dtype, int page_size, long long page_stride, long long pool_slots, void* cq, int cq_dtype, int tokens, int* status);
+int eg_latent_prepare(cudaStream_t stream, const float* down, long long ld, int q_rank, int rank, int rot, int rot_dims, int rot_half, const float* gain_q, const float* gain_c, float eps, const float* inv_freq, const int* positions, const int* slot_map, void* cache, int cache_dtype, int page_size, long long page_stride, long long pool_slots, void* cq, int cq_dtype, int tokens, int* status);
 // attention_latent.cu
-int eg_latent_absorb(cudaStream_t stream, int w_dtype, const float* q, long long ldq, const void* Uk, const int* positions, const float* inv_freq, int rot_dims, float scale, float* qa, int tokens, int heads, int dim, int rot, int rank);
+int eg_latent_absorb(cudaStream_t stream, int w_dtype, const float* q, long long ldq, const void* Uk, const int* positions, const float* inv_freq, int rot_dims, int rot_half, float scale, float* qa, int tokens, int heads, int dim, int rot, int rank);
 // attention_latent.cu
 int eg_attention_latent(cudaStream_t stream, int cache_dtype, const float* qa, const void* cache, const int* block_table, int table_stride, const int* token_seq, const int* positions, const float* sink, float* out, int tokens, int heads, int rank, int rot, int page_size, long long page_stride, int num_pages, int* status);
 // attention_latent.cu
 int eg_latent_expand(cudaStream_t stream, int w_dtype, const float* o, const void* Uv, void* out, int out_dtype, long long ldo, int tokens, int heads, int vdim, int rank);
 // moe.cu
-int eg_moe_route(cudaStream_t stream, int dtype, const void* h, long long ld, const float* router, const float* correction, const float* gate_w, float* logits, int* ids, float* weights, float* gate, int tokens, int width, int outputs, int top, int scoring);
+int eg_moe_route(cudaStream_t stream, int dtype, const void* h, long long ld, const float* router, const float* correction, const float* gate_w, float* logits, int* ids, float* weights, float* gate, int tokens, int width, int outputs, int top, int scoring, int groups, int keep, int normalize);
 // moe.cu
 int eg_moe_hidden(cudaStream_t stream, int dtype, const void* h, long long ld, const void* gate_up, const int* ids, const float* input_weights, void* act, int tokens, int width, int ff, int top, int experts, int activation, float limit);
 // moe.cu
@@ -88,7 +88,7 @@ int eg_attention_latent_mma_takes(int rank, int rot);
 // attention_latent_mma.cu
 int eg_attention_latent_mma(cudaStream_t stream, const void* qa, const void* cache, const int* block_table, int table_stride, const int* token_seq, const int* positions, const float* sink, void* out, float* part_o, float* part_ml, int tokens, int heads, int rank, int rot, int page_size, long long page_stride, int num_pages, int splits, int* status);
 // attention_latent_mma.cu
-int eg_latent_rotate_query(cudaStream_t stream, const void* q, long long ldq, const int* positions, const float* inv_freq, int rot_dims, float scale, void* qa, int tokens, int heads, int dim, int rot, int rank);
+int eg_latent_rotate_query(cudaStream_t stream, const void* q, long long ldq, const int* positions, const float* inv_freq, int rot_dims, int rot_half, float scale, void* qa, int tokens, int heads, int dim, int rot, int rank);
 // sandwich.cu
 int eg_token_shift(cudaStream_t stream, const float* rows, const float* mu, float* state, long long slot_floats, const int* token_seq, const int* seq_starts, const int* seq_slots, void* out, int out_dtype, int tokens, int hidden);
 // sandwich.cu
@@ -160,11 +160,11 @@ int eg_gemm_tcgen05_grouped_glu(cudaStream_t stream, const void* A, long long ld
 // attention_masked.cu
 int eg_masked_attention_prepare(cudaStream_t stream, int dtype, const float* proj, long long ld, const float* table, int rot_dims, float magnitude, const int* slot_map, void* k_cache, void* v_cache, int row_stride, long long head_stride, int page_size, long long page_stride, long long pool_slots, void* q_out, int tokens, int heads, int kv_heads, int maps, int dk, int dv, float norm_eps, const float* q_gain, const float* k_gain, int planes, int* status);
 // attention_masked.cu
-int eg_masked_attention(cudaStream_t stream, int dtype, const void* q, const void* k_cache, const void* v_cache, int row_stride, long long head_stride, const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* token_list, void* out, int out_dtype, long long ldo, int num_tokens, int heads, int kv_heads, int maps, int dk, int dv, int page_size, long long page_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, float out_scale, int planes, int* status);
+int eg_masked_attention(cudaStream_t stream, int dtype, const void* q, const void* k_cache, const void* v_cache, int row_stride, long long head_stride, const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* token_list, void* out, int out_dtype, long long ldo, int num_tokens, int heads, int kv_heads, int maps, int dk, int dv, int page_size, long long page_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, const float* slopes, float out_scale, int planes, int* status);
 // attention_paged.cu
-int eg_attention_paged_masked(cudaStream_t stream, const void* q, int ldq, const void* k_cache, const void* v_cache, const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* seq_context, void* out, int out_dtype, int ldo, float* partial_acc, float* partial_ml, int tokens, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, float out_scale, int splits, int* status, int* counters, int use_pdl, const int* token_list);
+int eg_attention_paged_masked(cudaStream_t stream, const void* q, int ldq, const void* k_cache, const void* v_cache, const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* seq_context, void* out, int out_dtype, int ldo, float* partial_acc, float* partial_ml, int tokens, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, const float* slopes, float out_scale, int splits, int* status, int* counters, int use_pdl, const int* token_list);
 // attention_paged.cu
-int eg_attention_prefill_masked(cudaStream_t stream, const void* q, int ldq, const void* k_cache, const void* v_cache, const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, void* out, int out_dtype, int ldo, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, float out_scale, int* status);
+int eg_attention_prefill_masked(cudaStream_t stream, const void* q, int ldq, const void* k_cache, const void* v_cache, const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, void* out, int out_dtype, int ldo, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale, float softcap, const float* sinks, const float* slopes, float out_scale, int* status);
 // attention_masked.cu
 int eg_attention_map_difference(cudaStream_t stream, const float* maps, void* out, int out_dtype, long long ldo, int tokens, int heads, int dv, float lambda, float eps, float post);
 // gated_delta.cu
@@ -182,11 +182,21 @@ int eg_gemm_tcgen05_pair_glu_bias(cudaStream_t stream, const void* A, long long 
 // sandwich.cu
 int eg_rmsnorm_add_rows(cudaStream_t stream, float* residual, const void* y, int y_dtype, long long ldy, const float* bias, const float* gain, float eps, void* out, int out_dtype, int tokens, int hidden);
 // attention_tcgen05.cu
-int eg_attention_prefill_tcgen05_masked(cudaStream_t stream, const void* q, long long ldq, int total_tokens, const void* k_cache, const void* v_cache, const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, void* out, int out_dtype, long long ldo, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale, const float* sinks, float out_scale, int* status, int max_parts, int part_tiles, float* partial_o, float* partial_ml, int* queue);
+int eg_attention_prefill_tcgen05_masked(cudaStream_t stream, const void* q, long long ldq, int total_tokens, const void* k_cache, const void* v_cache, const int* block_table, int table_stride, const int* positions, const int* tiles, int num_tiles, void* out, int out_dtype, long long ldo, int num_heads, int num_kv_heads, int maps, int head_dim, int page_size, long long page_stride, long long head_stride, int num_pages, int window, int chunk, int keep_first, float scale, const float* sinks, const float* slopes, float out_scale, int* status, int max_parts, int part_tiles, float* partial_o, float* partial_ml, int* queue);
 // norm.cu
 int eg_add_group_rmsnorm(cudaStream_t stream, int delta_dtype, int out_dtype, float* residual, const void* delta, const int* rows, const float* gain, void* out, int num_rows, int hidden, int groups, float eps);
 // embedding.cu
 int eg_add_waves(cudaStream_t stream, float* residual, const int* positions, const float* head, const float* tail, int tokens, int hidden);
+// embedding.cu
+int eg_embedding_rmsnorm(cudaStream_t stream, int dtype, const int* ids, const void* table, const float* gain, float eps, float* residual, int tokens, int hidden, int vocab, int* status);
+// activation.cu
+int eg_gelu(cudaStream_t stream, const void* x, int x_dtype, long long ldx, void* out, int out_dtype, long long ldo, int tokens, int n);
+// activation.cu
+int eg_sigmoid_gate(cudaStream_t stream, int dtype, void* values, long long ldv, const float* gate, long long ldg, int tokens, int n, int span);
+// gemm_skinny.cu
+int eg_gemm_skinny_gelu(cudaStream_t stream, int norm, int use_pdl, const void* W, long long ldw, int M, int N, int K, const void* x, long long ldx, const float* resid_in, float* resid_out, const void* delta, const float* gain, float eps, const float* ss_in, int ss_parts, void* out, long long ldo, int row_blocks, int k_slices, int k_split, float* scratch, int* counters, int* status);
+// gemm_tcgen05.cu
+int eg_gemm_tcgen05_pair_gelu(cudaStream_t stream, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int M, int N, int K, int tile_n, int* status);
 // sandwich.cu
 int eg_rmsnorm_pair(cudaStream_t stream, const float* a, const float* b, const float* gain_a, const float* gain_b, float eps, float factor, float* out, int tokens, int hidden);
 // attention_sigmoid.cu

@@ -180,6 +180,30 @@ public:
         return out;
     }
 
+    // out [M, out_features] (compute dtype) = gelu(input W^T) by the decode product, the input rows x or a norm in front
+    Rows skinny_gelu(const StepContext& ctx, int M, const Rows* x, const NormInFront* norm) const {
+        const int N = out_features;
+        const plans::SkinnyPlan plan = plans::skinny_plan(N, in_features, 0);
+        float* partials = nullptr;
+        int* counters = nullptr;
+        if (plan.k_split > 1) {
+            const size_t groups = (size_t)(N + plan.row_blocks * 16 - 1) / (plan.row_blocks * 16);
+            const size_t floats = (size_t)plan.k_split * groups * plan.row_blocks * 16 * plans::skinny_padded_tokens(M);
+            if (floats > KernelScratch::SKINNY_FLOATS || groups > KernelScratch::SKINNY_COUNTERS)
+                throw DeviceError("a decode product's split needs more scratch memory than the engine holds");
+            partials = ctx.scratch->skinny_partials.as<float>();
+            counters = ctx.scratch->skinny_counters.as<int>();
+        }
+        Rows out{ctx.take_rows(M, N, DType::BF16), DType::BF16, M, N, N};
+        const bool prepared = norm && norm->prepared_rows;
+        launch_check(eg_gemm_skinny_gelu(ctx.stream, norm ? (prepared ? 2 : 1) : 0, plans::use_pdl(), weight, in_features, M, N, in_features, x ? x->p : nullptr,
+                                         x ? x->ld : 0, norm ? norm->residual : nullptr, norm ? norm->residual_out : nullptr,
+                                         prepared ? norm->prepared_rows : norm ? norm->delta : nullptr, norm ? norm->gain : nullptr, norm ? norm->eps : 0.f,
+                                         norm ? norm->prepared_sums : nullptr, norm ? norm->prepared_parts : 0, out.p, N, plan.row_blocks, plan.k_slices,
+                                         plan.k_split, partials, counters, ctx.status), "gemm_skinny_gelu");
+        return out;
+    }
+
     // whether with_following_norm can run for this input (the decode kernel takes it)
     bool takes_following_norm(const Rows& x) const {
         return dtype == DType::BF16 && plans::gemm_skinny_takes(dtype, x.rows, in_features) && x.rows <= plans::FUSED_NORM_MAX_TOKENS && aligned(x);
@@ -845,19 +869,86 @@ private:
     Linear gate_up_, down_;
 };
 
+// ---- dense feed-forward without a gate: down(act(up h)), act the squared ReLU max(z, 0)^2 ("relu2") or the exact gelu
+// z / 2 (1 + erf(z / sqrt 2)) ("gelu").  Parameters: hidden_size, ff, activation.  Tensors: .up [ff, hidden], .down [hidden, ff] ---------
+class UngatedFeedForward : public FeedForward {
+public:
+    UngatedFeedForward(const Params& p, const std::string& prefix)
+        : FeedForward(p, prefix), hidden_((int)p.integer("hidden_size")), ff_((int)p.integer("ff")), gelu_(p.text("activation", "relu2") == "gelu") {
+        if (hidden_ <= 0 || ff_ <= 0) throw std::invalid_argument("a dense feed-forward's sizes must be positive");
+        if (!gelu_ && p.text("activation", "relu2") != "relu2") throw std::invalid_argument("an ungated feed-forward's activation is 'relu2' or 'gelu'");
+    }
+    std::vector<TensorRequest> tensor_requests() const override {
+        return {TensorRequest::matrix(prefix + ".up", ff_, hidden_), TensorRequest::matrix(prefix + ".down", hidden_, ff_)};
+    }
+    void load(const HostTensors& file, DType dtype) override {
+        up_ = Linear(need_tensor(file, prefix + ".up"), nullptr, dtype);
+        down_ = Linear(need_tensor(file, prefix + ".down"), nullptr, dtype);
+    }
+    size_t weight_bytes() const override { return up_.weight_bytes() + down_.weight_bytes(); }
+    size_t arena_bytes(long long T) const override { return (size_t)T * ((size_t)ff_ * 8 + (size_t)hidden_ * 4) + (1u << 16); }
+    bool capturable() const override { return true; }
+
+    Delta forward(const StepContext& ctx, PartInput in, const FollowingNorm*) override {
+        const int T = ctx.num_tokens;
+        const DType dtype = ctx.dtype;
+        const Rows h = in.pending ? in.pending->materialize() : in.rows;
+        Rows act;
+        if (plans::gemm_skinny_takes(dtype, T, hidden_) && Linear::aligned(h)) {
+            // steps of few tokens: the decode product with the activation on its finished sums
+            act = gelu_ ? up_.skinny_gelu(ctx, T, &h, nullptr) : up_.skinny_relu2(ctx, h);
+        } else if (plans::gemm_tcgen05_wide_takes(dtype, T, ff_, hidden_) && Linear::aligned(h)) {
+            // prompts: the product on the tcgen05 tensor cores (CTA pairs) with the activation in its epilogue
+            act = Rows{ctx.take_rows(T, ff_, dtype), dtype, T, ff_, ff_};
+            launch_check((gelu_ ? eg_gemm_tcgen05_pair_gelu : eg_gemm_tcgen05_pair_relu2)(ctx.stream, h.p, h.ld, up_.weight, hidden_, act.p, ff_, T, ff_, hidden_,
+                                                                                         256, ctx.status), "gemm_tcgen05_pair_act");
+        } else {
+            act = Rows{ctx.take_rows(T, ff_, dtype), dtype, T, ff_, ff_};
+            const Rows z = up_(ctx, h, /*out_f32=*/true);
+            launch_check((gelu_ ? eg_gelu : eg_squared_relu)(ctx.stream, z.p, (int)z.dtype, z.ld, act.p, (int)dtype, act.ld, T, ff_), "activation");
+        }
+        const Rows o = down_(ctx, act, /*out_f32=*/true);
+        Delta d;
+        d.p = o.p;
+        d.dtype = o.dtype;
+        return d;
+    }
+
+private:
+    int hidden_, ff_;
+    bool gelu_;
+    Linear up_, down_;
+};
+
 // ---- token embedding: residual[t] = E[id[t]] (src/models/embedding.cpp:54-76) ---------------------------------------
 class TokenEmbedding : public Embedding {
 public:
     TokenEmbedding(const Params& p, const std::string& prefix)
         : Embedding(p, prefix), vocab_((int)p.integer("vocab_size")), hidden_((int)p.integer("hidden_size")), weight_name_(prefix + p.text("weight_name", ".weight")),
-          scale_(p.has("scale") ? (float)p.real("scale") : 1.0f) {}
-    std::vector<TensorRequest> tensor_requests() const override { return {TensorRequest::matrix(weight_name_, vocab_, hidden_)}; }
+          scale_(p.has("scale") ? (float)p.real("scale") : 1.0f), norm_name_(p.has("norm_name") ? prefix + p.text("norm_name") : ""),
+          norm_eps_((float)p.real("norm_eps", 0.0)), norm_offset_((float)p.real("norm_offset", 0.0)) {
+        if (!norm_name_.empty() && scale_ != 1.0f) throw std::invalid_argument("a token embedding has a scale or a norm, not both");
+    }
+    std::vector<TensorRequest> tensor_requests() const override {
+        std::vector<TensorRequest> r = {TensorRequest::matrix(weight_name_, vocab_, hidden_)};
+        if (!norm_name_.empty()) r.push_back(TensorRequest::vector(norm_name_, hidden_).with_init(norm_offset_ != 0.f ? "zero" : "one"));
+        return r;
+    }
     void load(const HostTensors& file, DType dtype) override {
         table_ = upload(need_tensor(file, weight_name_), dtype);
         dtype_ = dtype;
+        if (norm_name_.empty()) return;
+        std::vector<float> g = host_floats(need_tensor(file, norm_name_));
+        for (float& v : g) v += norm_offset_;
+        norm_gain_ = upload(g.data(), g.size(), DType::F32);
     }
     bool capturable() const override { return true; }
     void forward(const StepContext& ctx, float* residual) override {
+        if (!norm_name_.empty()) {  // the stream starts as the RMS norm of the row
+            launch_check(eg_embedding_rmsnorm(ctx.stream, (int)dtype_, ctx.token_ids, table_.get(), norm_gain_.as<float>(), norm_eps_, residual, ctx.num_tokens,
+                                              hidden_, vocab_, ctx.status), "embedding_rmsnorm");
+            return;
+        }
         if (scale_ != 1.0f) {       // residual[t] = scale * E[id[t]]
             launch_check(eg_embedding_gather_scaled(ctx.stream, (int)dtype_, ctx.token_ids, table_.get(), residual, ctx.num_tokens, hidden_, vocab_, scale_,
                                                     ctx.status), "embedding_gather_scaled");
@@ -868,7 +959,7 @@ public:
     }
     const void* table() const override { return table_.get(); }
     bool fused_gather(const void** table, int* vocab) const override {
-        if (dtype_ != DType::BF16 || hidden_ % 4 || scale_ != 1.0f) return false;
+        if (dtype_ != DType::BF16 || hidden_ % 4 || scale_ != 1.0f || !norm_name_.empty()) return false;
         *table = table_.get();
         *vocab = vocab_;
         return true;
@@ -878,8 +969,10 @@ private:
     int vocab_, hidden_;
     std::string weight_name_;
     float scale_;                   // parameter scale: a factor on every embedding row (default 1)
+    std::string norm_name_;         // parameter norm_name (suffix): an RMS norm of every row, its gain norm_offset plus this tensor, norm_eps under the root
+    float norm_eps_, norm_offset_;
     DType dtype_ = DType::BF16;
-    DeviceBuffer table_;
+    DeviceBuffer table_, norm_gain_;
 };
 
 // ---- output head: logits = x E^T when tied (the reference always is, src/models/gpt_model.cpp:324-328,
@@ -947,6 +1040,11 @@ inline void register_builtin_parts() {
     if (r.mixers.count("attention")) return;
     r.mixers["attention"] = [](const Params& p, const std::string& prefix, std::shared_ptr<PositionEncoding> pos) {
         return std::make_shared<Attention>(p, prefix, std::move(pos));
+    };
+    r.feed_forwards["squared_relu"] = [](const Params& p, const std::string& prefix) { return std::make_shared<UngatedFeedForward>(p, prefix); };
+    r.feed_forwards["gelu"] = [](Params p, const std::string& prefix) {
+        p.set("activation", "gelu");
+        return std::make_shared<UngatedFeedForward>(p, prefix);
     };
     r.feed_forwards["swiglu"] = [](const Params& p, const std::string& prefix) { return std::make_shared<SwiGLU>(p, prefix); };
     r.norms["rmsnorm"] = [](const Params& p, const std::string& prefix) { return std::make_shared<RMSNorm>(p, prefix); };

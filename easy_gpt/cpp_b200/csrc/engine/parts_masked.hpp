@@ -13,7 +13,8 @@ namespace easygpt::engine {
 // `maps` keys of `dim` values and one value of `vdim` values:  q, k, v = W_q h, W_k h, W_v h as ONE product (rows stacked),
 // float32 out;  with qk_norm "unit" or "gain", q and k are divided by their root mean square per head and map (norm_eps under
 // the root) and, for "gain", multiplied by the tensors .q.norm / .k.norm [dim];  then they are turned by the layer's position
-// encoding (a half rotation over its first dimensions);  score = (q . k) * scale, with softcap c: c tanh(score / c);
+// encoding (a half rotation over its first dimensions);  score = (q . k) * scale, with softcap c: c tanh(score / c), with
+// slopes 1 minus 2^(-8 (h + 1) / H) times the distance p - j for head h;
 // position p sees j <= p with p - j < window (if given) and floor(j / chunk) = floor(p / chunk) (if given), and every
 // j < keep_first;  the softmax's denominator has one more term exp(sink_h) with `sinks` (tensor .sink [H]);
 // with maps = 2 and lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (tensors .lq1 .lk1 .lq2 .lk2 [dim]):
@@ -24,8 +25,11 @@ namespace easygpt::engine {
 // tcgen05 one for prompt portions of 33 tokens and more (heads of 64 and 128, no soft cap), the tiled mma.sync one for shorter
 // portions, heads of 32 and capped scores, the split-key one for single tokens; everything else runs on the generic kernel.  With a window
 // or a chunk the cache manager gives pages back that no coming token can see, except those of the kept first positions.
+// With own_keys 0 the layer projects queries only and reads the keys and values that another run entry cached (the same head counts
+// and sizes; mask, scale and all else its own); cached_back then says for all layers of such a family how far back any of them looks
+// (-1: all keys), which is what the cache keeps.
 // Parameters: hidden_size, heads, kv_heads, dim, vdim, scale, maps, window, chunk, keep_first, softcap, sinks, qk_norm,
-// norm_eps, diff, out_scale.  Tensors: .q .k .v .o (+ .q.norm .k.norm, .sink, .lq1 .lk1 .lq2 .lk2).
+// norm_eps, diff, out_scale, slopes, own_keys, cached_back.  Tensors: .q .k .v .o (+ .q.norm .k.norm, .sink, .lq1 .lk1 .lq2 .lk2).
 class MaskedAttention : public Mixer {
 public:
     MaskedAttention(const Params& p, const std::string& prefix, std::shared_ptr<PositionEncoding> position)
@@ -33,7 +37,7 @@ public:
           dk_((int)p.integer("dim")), dv_((int)p.integer("vdim")), maps_((int)p.integer("maps", 1)), scale_((float)p.real("scale")),
           window_(p.integer("window", 0)), chunk_(p.integer("chunk", 0)), keep_first_(p.integer("keep_first", 0)), softcap_((float)p.real("softcap", 0.0)),
           sinks_(p.integer("sinks", 0) != 0), norm_kind_(p.text("qk_norm", "none")), norm_eps_((float)p.real("norm_eps", 0.0)), diff_(p.real("diff", 0.0)),
-          out_scale_((float)p.real("out_scale", 1.0)) {
+          out_scale_((float)p.real("out_scale", 1.0)), sloped_(p.integer("slopes", 0) != 0), own_keys_(p.integer("own_keys", 1) != 0) {
         if (hidden_ <= 0 || heads_ <= 0 || kv_heads_ <= 0 || dk_ <= 0 || dv_ <= 0) throw std::invalid_argument("masked attention: sizes must be positive");
         if (heads_ % kv_heads_) throw std::invalid_argument("masked attention: heads must be a multiple of kv_heads");
         if (maps_ != 1 && maps_ != 2) throw std::invalid_argument("masked attention: a head has one map, or two of which the second is taken off the first");
@@ -45,12 +49,14 @@ public:
     }
     std::vector<TensorRequest> tensor_requests() const override {
         std::vector<TensorRequest> r = {TensorRequest::matrix(prefix + ".q", (long long)heads_ * maps_ * dk_, hidden_),
-                                        TensorRequest::matrix(prefix + ".k", (long long)kv_heads_ * maps_ * dk_, hidden_),
-                                        TensorRequest::matrix(prefix + ".v", (long long)kv_heads_ * dv_, hidden_),
                                         TensorRequest::matrix(prefix + ".o", hidden_, (long long)heads_ * dv_)};
+        if (own_keys_) {
+            r.push_back(TensorRequest::matrix(prefix + ".k", (long long)kv_heads_ * maps_ * dk_, hidden_));
+            r.push_back(TensorRequest::matrix(prefix + ".v", (long long)kv_heads_ * dv_, hidden_));
+        }
         if (norm_kind_ == "gain") {
             r.push_back(TensorRequest::vector(prefix + ".q.norm", dk_).with_init("one"));
-            r.push_back(TensorRequest::vector(prefix + ".k.norm", dk_).with_init("one"));
+            if (own_keys_) r.push_back(TensorRequest::vector(prefix + ".k.norm", dk_).with_init("one"));
         }
         if (sinks_) r.push_back(TensorRequest::vector(prefix + ".sink", heads_).with_init("zero"));
         if (maps_ == 2)
@@ -60,14 +66,20 @@ public:
     void load(const HostTensors& file, DType dtype) override {
         std::vector<float> w;
         for (const char* n : {".q", ".k", ".v"}) {
+            if (!own_keys_ && n != std::string(".q")) continue;
             const std::vector<float> part = host_floats(need_tensor(file, prefix + n));
             w.insert(w.end(), part.begin(), part.end());
         }
-        qkv_ = Linear(w.data(), (heads_ + kv_heads_) * maps_ * dk_ + kv_heads_ * dv_, hidden_, nullptr, dtype);
+        qkv_ = Linear(w.data(), heads_ * maps_ * dk_ + (own_keys_ ? kv_heads_ * (maps_ * dk_ + dv_) : 0), hidden_, nullptr, dtype);
         out_ = Linear(need_tensor(file, prefix + ".o"), nullptr, dtype);
         if (norm_kind_ == "gain") {
             q_gain_ = upload_f32(file, prefix + ".q.norm");
-            k_gain_ = upload_f32(file, prefix + ".k.norm");
+            if (own_keys_) k_gain_ = upload_f32(file, prefix + ".k.norm");
+        }
+        if (sloped_) {
+            std::vector<float> s((size_t)heads_ * maps_);
+            for (size_t r = 0; r < s.size(); ++r) s[r] = (float)std::exp2(-8.0 * (double)(r / maps_ + 1) / heads_);
+            slopes_ = upload(s.data(), s.size(), DType::F32);
         }
         if (sinks_) sink_ = upload_f32(file, prefix + ".sink");
         if (maps_ == 2) {
@@ -96,7 +108,8 @@ public:
         return window_ > 0 ? window_ : chunk_ > 0 ? chunk_ : -1;
     }
     CacheNeed cache_need() const override {
-        const CacheNeed n = planes() ? CacheNeed::paged(kv_heads_ * maps_, dk_, kept_back()) : CacheNeed::paged_joint(kv_heads_, maps_ * dk_, dv_, kept_back());
+        const long long back = params.has("cached_back") ? params.integer("cached_back") : kept_back();
+        const CacheNeed n = planes() ? CacheNeed::paged(kv_heads_ * maps_, dk_, back) : CacheNeed::paged_joint(kv_heads_, maps_ * dk_, dv_, back);
         return n.keeping_first(keep_first_);
     }
 
@@ -104,6 +117,7 @@ public:
         const int T = ctx.num_tokens;
         const DType dtype = ctx.dtype;
         if (cache.group < 0) throw DeviceError("masked attention was handed no paged cache");
+        if (cache.writes && !own_keys_) throw DeviceError("masked attention without keys of its own reads another entry's cache");
         const GroupTables& tables = ctx.groups.at(cache.group);
         const Rows h = in.pending ? in.pending->materialize() : in.rows;
         const Rows proj = qkv_(ctx, h, /*out_f32=*/true);
@@ -121,7 +135,7 @@ public:
                                                  tables.slot_map, cache.writes ? cache.k : nullptr, values, row_stride, cache.head_stride, cache.page_size,
                                                  cache.page_stride, (long long)cache.num_pages * cache.page_size, q.p, T, heads_, kv_heads_, maps_, dk_, dv_,
                                                  norm_kind_ == "none" ? -1.f : norm_eps_, norm_kind_ == "gain" ? q_gain_.as<float>() : nullptr,
-                                                 norm_kind_ == "gain" ? k_gain_.as<float>() : nullptr, planes() ? 1 : 0, ctx.status), "masked_attention_prepare");
+                                                 norm_kind_ == "gain" && own_keys_ ? k_gain_.as<float>() : nullptr, planes() ? 1 : 0, ctx.status), "masked_attention_prepare");
         Rows attn{ctx.take_rows(T, heads_ * dv_, dtype), dtype, T, heads_ * dv_, heads_ * dv_};
         // one map: the heads' outputs at once; two: both maps of every head in float32, then their difference, its norm and its
         // factor in one kernel
@@ -129,14 +143,14 @@ public:
         void* out = both ? (void*)both : attn.p;
         const DType out_dtype = both ? DType::F32 : dtype;
         const long long ldo = both ? (long long)rows * dv_ : attn.ld;
-        const float* sinks = sinks_ ? sink_.as<float>() : nullptr;
+        const float *sinks = sinks_ ? sink_.as<float>() : nullptr, *slopes = sloped_ ? slopes_.as<float>() : nullptr;
         const float factor = both ? 1.0f : out_scale_;
         if (dtype == DType::BF16 && planes() && (dk_ == 32 || dk_ == 64 || dk_ == 128) && cache.page_size % 16 == 0) {
             auto tiled = [&](const int* tiles, int count) {
                 launch_check(eg_attention_prefill_masked(ctx.stream, q.p, (int)q.ld, cache.k, cache.v, tables.block_table, tables.table_width, ctx.positions, tiles,
                                                          count, out, (int)out_dtype, (int)ldo, rows, kv_heads_ * maps_, maps_, dk_, cache.page_size, cache.page_stride,
                                                          cache.head_stride, cache.num_pages, (int)window_, (int)chunk_, (int)keep_first_, scale_, softcap_, sinks,
-                                                         factor, ctx.status), "attention_prefill_masked");
+                                                         slopes, factor, ctx.status), "attention_prefill_masked");
             };
             // prompt portions in tiles of query tokens, on tcgen05 when they are long enough to fill its 128-row tiles; single
             // tokens (decoding, short entries) split over their keys
@@ -159,7 +173,7 @@ public:
                 launch_check(eg_attention_prefill_tcgen05_masked(ctx.stream, q.p, q.ld, T, cache.k, cache.v, tables.block_table, tables.table_width, ctx.positions,
                                                                  ctx.query_tiles, ctx.num_tiles, out, (int)out_dtype, ldo, rows, key_heads, maps_, dk_, cache.page_size,
                                                                  cache.page_stride, cache.head_stride, cache.num_pages, (int)window_, (int)chunk_, (int)keep_first_,
-                                                                 scale_, sinks, factor, ctx.status, parts, part_tiles, partial_o, partial_ml,
+                                                                 scale_, sinks, slopes, factor, ctx.status, parts, part_tiles, partial_o, partial_ml,
                                                                  ctx.scratch->prefill_queue.as<int>()), "attention_prefill_tcgen05_masked");
             } else if (ctx.query_tiles) {
                 tiled(ctx.query_tiles, ctx.num_tiles);
@@ -179,13 +193,13 @@ public:
                 launch_check(eg_attention_paged_masked(ctx.stream, q.p, (int)q.ld, cache.k, cache.v, tables.block_table, tables.table_width, ctx.token_seq,
                                                        ctx.positions, ctx.query_tiles ? nullptr : ctx.seq_context, out, (int)out_dtype, (int)ldo, acc, ml, singles,
                                                        rows, key_heads, maps_, dk_, cache.page_size, cache.page_stride, cache.head_stride, cache.num_pages,
-                                                       (int)window_, (int)chunk_, (int)keep_first_, scale_, softcap_, sinks, factor, splits, ctx.status, counters,
+                                                       (int)window_, (int)chunk_, (int)keep_first_, scale_, softcap_, sinks, slopes, factor, splits, ctx.status, counters,
                                                        plans::use_pdl(), ctx.query_tiles ? ctx.small_tokens : nullptr), "attention_paged_masked");
             }
         } else {
             launch_check(eg_masked_attention(ctx.stream, (int)dtype, q.p, cache.k, values, row_stride, cache.head_stride, tables.block_table, tables.table_width,
                                              ctx.token_seq, ctx.positions, nullptr, out, (int)out_dtype, ldo, T, heads_, kv_heads_, maps_, dk_, dv_, cache.page_size,
-                                             cache.page_stride, cache.num_pages, (int)window_, (int)chunk_, (int)keep_first_, scale_, softcap_, sinks, factor,
+                                             cache.page_stride, cache.num_pages, (int)window_, (int)chunk_, (int)keep_first_, scale_, softcap_, sinks, slopes, factor,
                                              planes() ? 1 : 0, ctx.status), "masked_attention");
         }
         if (both)
@@ -208,8 +222,9 @@ private:
     float norm_eps_;
     double diff_;
     float out_scale_, lambda_ = 0.f;
+    bool sloped_, own_keys_;
     Linear qkv_, out_;
-    DeviceBuffer q_gain_, k_gain_, sink_;
+    DeviceBuffer q_gain_, k_gain_, sink_, slopes_;
 };
 
 // ---- gated delta rule with a decay per key channel ---------------------------------------------------------------------------

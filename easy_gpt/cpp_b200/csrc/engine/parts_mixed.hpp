@@ -1,6 +1,6 @@
 // Further parts: a gain per channel on a branch's output (a layer scale), a causal convolution over time in front of a
 // mixer, attention whose scores are mixed across the heads before the softmax and whose values are the keys as projected,
-// a dense feed-forward with a squared ReLU, and a small gated map of a per-token vector that joins the stream through a norm
+// and a small gated map of a per-token vector that joins the stream through a norm
 // of its own.  Each takes its sizes, constants and tensor-name suffixes from its parameters and knows nothing of the model
 // around it.
 #pragma once
@@ -193,53 +193,6 @@ private:
     DeviceBuffer q_weight_, k_weight_, mix_;
 };
 
-// ---- dense feed-forward with a squared ReLU: down(max(up h, 0)^2).  Parameters: hidden_size, ff.  Tensors: .up [ff, hidden],
-// .down [hidden, ff] ---------------------------------------------------------------------------------------------------------------
-class SquaredReluFeedForward : public FeedForward {
-public:
-    SquaredReluFeedForward(const Params& p, const std::string& prefix) : FeedForward(p, prefix), hidden_((int)p.integer("hidden_size")), ff_((int)p.integer("ff")) {
-        if (hidden_ <= 0 || ff_ <= 0) throw std::invalid_argument("a dense feed-forward's sizes must be positive");
-    }
-    std::vector<TensorRequest> tensor_requests() const override {
-        return {TensorRequest::matrix(prefix + ".up", ff_, hidden_), TensorRequest::matrix(prefix + ".down", hidden_, ff_)};
-    }
-    void load(const HostTensors& file, DType dtype) override {
-        up_ = Linear(need_tensor(file, prefix + ".up"), nullptr, dtype);
-        down_ = Linear(need_tensor(file, prefix + ".down"), nullptr, dtype);
-    }
-    size_t weight_bytes() const override { return up_.weight_bytes() + down_.weight_bytes(); }
-    size_t arena_bytes(long long T) const override { return (size_t)T * ((size_t)ff_ * 8 + (size_t)hidden_ * 4) + (1u << 16); }
-    bool capturable() const override { return true; }
-
-    Delta forward(const StepContext& ctx, PartInput in, const FollowingNorm*) override {
-        const int T = ctx.num_tokens;
-        const DType dtype = ctx.dtype;
-        const Rows h = in.pending ? in.pending->materialize() : in.rows;
-        Rows act;
-        if (plans::gemm_skinny_takes(dtype, T, hidden_) && Linear::aligned(h)) {
-            // steps of few tokens: the decode product with the square on its finished sums
-            act = up_.skinny_relu2(ctx, h);
-        } else if (plans::gemm_tcgen05_wide_takes(dtype, T, ff_, hidden_) && Linear::aligned(h)) {
-            // prompts: the product on the tcgen05 tensor cores (CTA pairs) with the activation in its epilogue
-            act = Rows{ctx.take_rows(T, ff_, dtype), dtype, T, ff_, ff_};
-            launch_check(eg_gemm_tcgen05_pair_relu2(ctx.stream, h.p, h.ld, up_.weight, hidden_, act.p, ff_, T, ff_, hidden_, 256, ctx.status), "gemm_tcgen05_pair_relu2");
-        } else {
-            act = Rows{ctx.take_rows(T, ff_, dtype), dtype, T, ff_, ff_};
-            const Rows z = up_(ctx, h, /*out_f32=*/true);
-            launch_check(eg_squared_relu(ctx.stream, z.p, (int)z.dtype, z.ld, act.p, (int)dtype, act.ld, T, ff_), "squared_relu");
-        }
-        const Rows o = down_(ctx, act, /*out_f32=*/true);
-        Delta d;
-        d.p = o.p;
-        d.dtype = o.dtype;
-        return d;
-    }
-
-private:
-    int hidden_, ff_;
-    Linear up_, down_;
-};
-
 // ---- a per-layer token input ------------------------------------------------------------------------------------------------
 // Every token brings a vector e of `side` values of its own, the columns [column, column + side) of a table [vocab, columns]
 // that all layers share.  It is gated by the stream and mapped to the model's width:
@@ -317,7 +270,6 @@ inline void register_mixed_parts() {
     r.mixers["mixed_attention"] = [](const Params& p, const std::string& prefix, std::shared_ptr<PositionEncoding> pos) {
         return std::make_shared<MixedAttention>(p, prefix, std::move(pos));
     };
-    r.feed_forwards["squared_relu"] = [](const Params& p, const std::string& prefix) { return std::make_shared<SquaredReluFeedForward>(p, prefix); };
     r.feed_forwards["token_side"] = [](const Params& p, const std::string& prefix) { return std::make_shared<TokenSide>(p, prefix); };
 }
 

@@ -117,19 +117,22 @@ private:
 //   c_q = unit_rms(W_dq h) * g_q;  q = W_uq c_q, head by head (dim plain | rot_dim rotated)
 //   (c' | k_r') = W_dkv h;  c = unit_rms(c') * g_kv [kv_rank];  k_r = rotate(k_r') [rot_dim], one for all heads
 //   key_h = (W_uk,h c | k_r), value_h = W_uv,h c;  score = (q_plain . key_plain + rotate(q_rot) . k_r) * scale
-//   causal softmax whose denominator also holds exp(sink_h) if the model has sinks;  out = W_o (heads' values side by side)
-// Only (c | k_r) is cached: one row per token for all heads (CacheNeed::paged_rows).  The rotation turns neighbouring
-// pairs (2i, 2i+1) of the first rot_dims values by position * base^(-2i / rot_dims).
-// Parameters: hidden_size, heads, dim, rot_dim, vdim, kv_rank, q_rank, scale, rot_base, rot_dims, eps, sink.
+//   causal softmax whose denominator also holds exp(sink_h) if the model has sinks;  out = W_o (heads' values side by side),
+//   with `gate` "values" or "heads" each value or each head times sigmoid(W_g h) first
+// Only (c | k_r) is cached: one row per token for all heads (CacheNeed::paged_rows).  The rotation turns pairs of
+// the first rot_dims values by position * base^(-2i / rot_dims): neighbours (2i, 2i+1), or with rot_layout "half" (i, i + rot_dims/2).
+// Parameters: hidden_size, heads, dim, rot_dim, vdim, kv_rank, q_rank, scale, rot_base, rot_dims, rot_layout, eps, sink, gate.
 // Tensors: .dq [q_rank, hidden], .dq.norm, .uq [H (dim + rot_dim), q_rank], .dkv [kv_rank + rot_dim, hidden], .dkv.norm,
-// .uk [H dim, kv_rank], .uv [H vdim, kv_rank], .sink [H], .o [hidden, H vdim].
+// .uk [H dim, kv_rank], .uv [H vdim, kv_rank], .sink [H], .g [H vdim or H, hidden], .o [hidden, H vdim].
 class LatentAttention : public Mixer {
 public:
     LatentAttention(const Params& p, const std::string& prefix, std::shared_ptr<PositionEncoding> position)
         : Mixer(p, prefix, std::move(position)), hidden_((int)p.integer("hidden_size")), heads_((int)p.integer("heads")), dim_((int)p.integer("dim")),
           rot_((int)p.integer("rot_dim")), vdim_((int)p.integer("vdim")), rank_((int)p.integer("kv_rank")), q_rank_((int)p.integer("q_rank")),
           rot_dims_((int)p.integer("rot_dims", p.integer("rot_dim"))), scale_((float)p.real("scale")), base_(p.real("rot_base")), eps_((float)p.real("eps")),
-          sink_(p.flag("sink", false)) {
+          sink_(p.flag("sink", false)), rot_half_(p.text("rot_layout", "interleaved") == "half"), gate_(p.text("gate", "none")) {
+        if (!rot_half_ && p.text("rot_layout", "interleaved") != "interleaved") throw std::invalid_argument("latent attention: rot_layout is 'interleaved' or 'half'");
+        if (gate_ != "none" && gate_ != "values" && gate_ != "heads") throw std::invalid_argument("latent attention: gate is 'none', 'values' or 'heads'");
         if (heads_ <= 0 || dim_ < 0 || rot_ < 0 || dim_ + rot_ <= 0 || vdim_ <= 0 || rank_ <= 0 || q_rank_ <= 0)
             throw std::invalid_argument("latent attention: sizes must be positive");
         if (rot_dims_ % 2 || rot_dims_ < 0 || rot_dims_ > rot_) throw std::invalid_argument("latent attention: rot_dims must be even and within rot_dim");
@@ -143,14 +146,21 @@ public:
                                         TensorRequest::matrix(prefix + ".uk", (long long)heads_ * dim_, rank_),
                                         TensorRequest::matrix(prefix + ".uv", (long long)heads_ * vdim_, rank_), TensorRequest::matrix(prefix + ".o", hidden_, (long long)heads_ * vdim_)};
         if (sink_) r.push_back(TensorRequest::vector(prefix + ".sink", heads_).with_init("zero"));
+        if (gates() > 0) r.push_back(TensorRequest::matrix(prefix + ".g", gates(), hidden_));
         return r;
     }
+    // logits of the output gate per token
+    int gates() const { return gate_ == "values" ? heads_ * vdim_ : gate_ == "heads" ? heads_ : 0; }
     void load(const HostTensors& file, DType dtype) override {
-        // one product for both down-projections: rows (query latent | latent | rotated key part)
+        // one product for everything that reads the layer's input: rows (query latent | latent | rotated key part | gate)
         std::vector<float> w = host_floats(need_tensor(file, prefix + ".dq"));
         const std::vector<float> dkv = host_floats(need_tensor(file, prefix + ".dkv"));
         w.insert(w.end(), dkv.begin(), dkv.end());
-        down_ = Linear(w.data(), q_rank_ + rank_ + rot_, hidden_, nullptr, dtype);
+        if (gates() > 0) {
+            const std::vector<float> g = host_floats(need_tensor(file, prefix + ".g"));
+            w.insert(w.end(), g.begin(), g.end());
+        }
+        down_ = Linear(w.data(), q_rank_ + rank_ + rot_ + gates(), hidden_, nullptr, dtype);
         up_q_ = Linear(need_tensor(file, prefix + ".uq"), nullptr, dtype);
         out_ = Linear(need_tensor(file, prefix + ".o"), nullptr, dtype);
         up_k_ = upload(need_tensor(file, prefix + ".uk"), dtype);
@@ -170,7 +180,7 @@ public:
         return down_.weight_bytes() + up_q_.weight_bytes() + out_.weight_bytes() + (size_t)heads_ * (dim_ + vdim_) * rank_ * dtype_size(down_.dtype);
     }
     size_t arena_bytes(long long T) const override {
-        const size_t per_token = (size_t)(q_rank_ + rank_ + rot_) * 4 + (size_t)q_rank_ * 4 + (size_t)heads_ * (dim_ + rot_) * 4 + (size_t)heads_ * (rank_ + rot_) * 4 +
+        const size_t per_token = (size_t)(q_rank_ + rank_ + rot_ + gates()) * 4 + (size_t)q_rank_ * 4 + (size_t)heads_ * (dim_ + rot_) * 4 + (size_t)heads_ * (rank_ + rot_) * 4 +
                                  (size_t)heads_ * rank_ * 4 + (size_t)heads_ * vdim_ * 4 + (size_t)hidden_ * 4;
         // the parts of an attention whose keys are cut: at most two CTAs an SM's worth of them beyond one per token
         const size_t parts = (size_t)(4 * plans::sm_count() + 64) * 16 * (size_t)(rank_ + 2) * 4;
@@ -187,10 +197,21 @@ public:
         const Rows h = in.pending ? in.pending->materialize() : in.rows;
         const Rows down = down_(ctx, h, /*out_f32=*/true);
         Rows cq{ctx.take_rows(T, q_rank_, dtype), dtype, T, q_rank_, q_rank_};
-        launch_check(eg_latent_prepare(ctx.stream, (const float*)down.p, down.ld, q_rank_, rank_, rot_, rot_dims_, gain_q_.as<float>(), gain_c_.as<float>(), eps_,
+        launch_check(eg_latent_prepare(ctx.stream, (const float*)down.p, down.ld, q_rank_, rank_, rot_, rot_dims_, rot_half_, gain_q_.as<float>(), gain_c_.as<float>(), eps_,
                                        inv_freq_.as<float>(), ctx.positions, tables.slot_map, cache.writes ? cache.k : nullptr, (int)dtype, cache.page_size,
                                        cache.page_stride, (long long)cache.num_pages * cache.page_size, cq.p, (int)dtype, T, ctx.status), "latent_prepare");
         const int D = rank_ + rot_;
+        // the heads' values side by side, through their gate and W_o
+        auto finish = [&](const Rows& values) {
+            if (gates() > 0)
+                launch_check(eg_sigmoid_gate(ctx.stream, (int)dtype, values.p, values.ld, (const float*)down.p + q_rank_ + rank_ + rot_, down.ld, T, heads_ * vdim_,
+                                             heads_ * vdim_ / gates()), "sigmoid_gate");
+            const Rows res = out_(ctx, values, /*out_f32=*/true);
+            Delta d;
+            d.p = res.p;
+            d.dtype = res.dtype;
+            return d;
+        };
         if (dtype == DType::BF16 && eg_attention_latent_mma_takes(rank_, rot_) && (dim_ + rot_) % 8 == 0 && dim_ % 8 == 0 && vdim_ % 8 == 0 && dim_ > 0) {
             // bfloat16 on the tensor cores: the per-head maps are strided batches of the library's product (a head is a
             // stride in the row, not a copy), the attention takes the heads of a token as the rows of its products
@@ -198,7 +219,7 @@ public:
             void* qa = ctx.take_rows((size_t)T * heads_, D, dtype);
             ctx.blas->gemm_bf16_batched(ctx.stream, false, rank_, T, dim_, scale_, up_k_.get(), rank_, (long long)dim_ * rank_, q.p, q.ld, dim_ + rot_, qa,
                                         (long long)heads_ * D, D, false, heads_);
-            launch_check(eg_latent_rotate_query(ctx.stream, q.p, q.ld, ctx.positions, inv_freq_.as<float>(), rot_dims_, scale_, qa, T, heads_, dim_, rot_, rank_),
+            launch_check(eg_latent_rotate_query(ctx.stream, q.p, q.ld, ctx.positions, inv_freq_.as<float>(), rot_dims_, rot_half_, scale_, qa, T, heads_, dim_, rot_, rank_),
                          "latent_rotate_query");
             const int splits = plans::latent_attention_splits(T, heads_, ctx.max_context_len);
             float *part_o = nullptr, *part_ml = nullptr;
@@ -213,15 +234,11 @@ public:
             Rows values{ctx.take_rows(T, heads_ * vdim_, dtype), dtype, T, heads_ * vdim_, heads_ * vdim_};
             ctx.blas->gemm_bf16_batched(ctx.stream, true, vdim_, T, rank_, 1.0f, up_v_.get(), rank_, (long long)vdim_ * rank_, o, (long long)heads_ * rank_, rank_,
                                         values.p, values.ld, vdim_, false, heads_);
-            const Rows res = out_(ctx, values, /*out_f32=*/true);
-            Delta d;
-            d.p = res.p;
-            d.dtype = res.dtype;
-            return d;
+            return finish(values);
         }
         const Rows q = up_q_(ctx, cq, /*out_f32=*/true);
         float* qa = ctx.take<float>((size_t)T * heads_ * (rank_ + rot_));
-        launch_check(eg_latent_absorb(ctx.stream, (int)dtype, (const float*)q.p, q.ld, up_k_.get(), ctx.positions, inv_freq_.as<float>(), rot_dims_, scale_, qa, T,
+        launch_check(eg_latent_absorb(ctx.stream, (int)dtype, (const float*)q.p, q.ld, up_k_.get(), ctx.positions, inv_freq_.as<float>(), rot_dims_, rot_half_, scale_, qa, T,
                                       heads_, dim_, rot_, rank_), "latent_absorb");
         float* o = ctx.take<float>((size_t)T * heads_ * rank_);
         launch_check(eg_attention_latent(ctx.stream, (int)dtype, qa, cache.k, tables.block_table, tables.table_width, ctx.token_seq, ctx.positions,
@@ -229,11 +246,7 @@ public:
                                          ctx.status), "attention_latent");
         Rows values{ctx.take_rows(T, heads_ * vdim_, dtype), dtype, T, heads_ * vdim_, heads_ * vdim_};
         launch_check(eg_latent_expand(ctx.stream, (int)dtype, o, up_v_.get(), values.p, (int)dtype, values.ld, T, heads_, vdim_, rank_), "latent_expand");
-        const Rows res = out_(ctx, values, /*out_f32=*/true);
-        Delta d;
-        d.p = res.p;
-        d.dtype = res.dtype;
-        return d;
+        return finish(values);
     }
 
 private:
@@ -241,7 +254,8 @@ private:
     float scale_;
     double base_;
     float eps_;
-    bool sink_;
+    bool sink_, rot_half_;
+    std::string gate_;
     Linear down_, up_q_, out_;
     DeviceBuffer up_k_, up_v_, gain_q_, gain_c_, sinks_, inv_freq_;
 };
@@ -259,23 +273,33 @@ private:
 // the softmax); correction 0 (no .correction tensor); activation "clamped" with limit (an expert is
 // down(g sigmoid(1.702 g) (u + 1)), g = min(gate x, limit), u = clamp(up x, -limit, limit)); weight_input 1 (the weight
 // multiplies the expert's input, out = sum of expert(weight * h), not its output); shared_gated 0 (the shared expert is added
-// as it is, no .shared.sg), shared_activation / shared_limit (the shared expert's own form).
+// as it is, no .shared.sg), shared_activation / shared_limit (the shared expert's own form); activation "gelu" (experts and shared
+// expert without a gate, down(gelu(up h)), the exact gelu; no .gate tensors); groups > 1 with keep_groups (the outputs form equal runs
+// of neighbours, a run counts the sum of its two largest s + correction, only the best keep_groups runs can be chosen); normalize 1
+// (the chosen weights are divided by their sum).
 class RoutedExperts : public FeedForward {
 public:
     RoutedExperts(const Params& p, const std::string& prefix)
         : FeedForward(p, prefix), hidden_((int)p.integer("hidden_size")), experts_((int)p.integer("experts")), identity_((int)p.integer("identity", 0)),
           top_((int)p.integer("top")), ff_((int)p.integer("ff", 0)), shared_ff_((int)p.integer("shared_ff", 0)),
           sigmoid_(p.text("scoring", "softmax") == "sigmoid"), corrected_(p.integer("correction", 1) != 0), clamped_(p.text("activation", "swiglu") == "clamped"),
-          weight_input_(p.integer("weight_input", 0) != 0), shared_gated_(p.integer("shared_gated", 1) != 0), limit_((float)p.real("limit", 0.0)) {
+          weight_input_(p.integer("weight_input", 0) != 0), shared_gated_(p.integer("shared_gated", 1) != 0), gated_(p.text("activation", "swiglu") != "gelu"),
+          groups_((int)p.integer("groups", 1)), keep_groups_((int)p.integer("keep_groups", p.integer("groups", 1))), normalize_(p.integer("normalize", 0) != 0),
+          limit_((float)p.real("limit", 0.0)) {
         if (p.text("scoring", "softmax") != "softmax" && !sigmoid_) throw std::invalid_argument("a routed feed-forward's scoring is 'softmax' or 'sigmoid'");
-        if (p.text("activation", "swiglu") != "swiglu" && !clamped_) throw std::invalid_argument("a routed feed-forward's activation is 'swiglu' or 'clamped'");
+        if (p.text("activation", "swiglu") != "swiglu" && !clamped_ && gated_) throw std::invalid_argument("a routed feed-forward's activation is 'swiglu', 'clamped' or 'gelu'");
         if (clamped_ && !(limit_ > 0.f)) throw std::invalid_argument("a clamped gate needs a positive limit");
         if (weight_input_ && identity_ > 0) throw std::invalid_argument("identity outputs take their weight on the output");
         if (experts_ < 0 || identity_ < 0 || experts_ + identity_ <= 0) throw std::invalid_argument("a routed feed-forward needs at least one router output");
         if (top_ < 1 || top_ > experts_ + identity_) throw std::invalid_argument("a routed feed-forward chooses between 1 and all of its router outputs");
+        if (groups_ < 1 || (experts_ + identity_) % groups_ || keep_groups_ < 1 || keep_groups_ > groups_)
+            throw std::invalid_argument("a routed feed-forward's groups must divide its router outputs, and between 1 and all of them are kept");
+        if (top_ > (experts_ + identity_) / groups_ * keep_groups_) throw std::invalid_argument("a routed feed-forward cannot choose more outputs than its kept groups have");
         if (experts_ > 0 && ff_ <= 0) throw std::invalid_argument("a routed feed-forward's experts need a positive ff");
         if (experts_ + identity_ > 2048) throw std::invalid_argument("a routed feed-forward takes at most 2048 router outputs");
-        if (shared_ff_ > 0) {
+        if (shared_ff_ > 0 && !gated_) {
+            shared_ = std::make_shared<UngatedFeedForward>(Params{{"hidden_size", hidden_}, {"ff", shared_ff_}, {"activation", "gelu"}}, prefix + ".shared");
+        } else if (shared_ff_ > 0) {
             Params sp{{"hidden_size", hidden_}, {"intermediate_size", shared_ff_}, {"gate_name", ".gate"}, {"up_name", ".up"}, {"down_name", ".down"}};
             if (p.has("shared_activation")) sp.set("activation", p.text("shared_activation"));
             if (p.has("shared_limit")) sp.set("limit", p.real("shared_limit"));
@@ -287,7 +311,7 @@ public:
         if (corrected_) r.push_back(TensorRequest::vector(prefix + ".correction", experts_ + identity_).with_init("zero"));
         for (int e = 0; e < experts_; ++e) {
             const std::string ep = prefix + ".e" + std::to_string(e);
-            r.push_back(TensorRequest::matrix(ep + ".gate", ff_, hidden_));
+            if (gated_) r.push_back(TensorRequest::matrix(ep + ".gate", ff_, hidden_));
             r.push_back(TensorRequest::matrix(ep + ".up", ff_, hidden_));
             r.push_back(TensorRequest::matrix(ep + ".down", hidden_, ff_));
         }
@@ -304,14 +328,17 @@ public:
         };
         router_ = f32(".router");
         if (corrected_) correction_ = f32(".correction");
-        // all experts in one block each: gate and up rows interleaved per hidden unit (gate_f, up_f), and the down maps
-        std::vector<float> gu((size_t)experts_ * 2 * ff_ * hidden_), dn((size_t)experts_ * hidden_ * ff_);
+        // all experts in one block each: gate and up rows interleaved per hidden unit (gate_f, up_f), or the up rows; and the down maps
+        const int first_rows = first_product_rows();
+        std::vector<float> gu((size_t)experts_ * first_rows * hidden_), dn((size_t)experts_ * hidden_ * ff_);
         for (int e = 0; e < experts_; ++e) {
             const std::string ep = prefix + ".e" + std::to_string(e);
-            const std::vector<float> g = host_floats(need_tensor(file, ep + ".gate")), u = host_floats(need_tensor(file, ep + ".up")),
-                                     d = host_floats(need_tensor(file, ep + ".down"));
-            float* base = gu.data() + (size_t)e * 2 * ff_ * hidden_;
-            for (int f = 0; f < ff_; ++f) {
+            const std::vector<float> u = host_floats(need_tensor(file, ep + ".up")), d = host_floats(need_tensor(file, ep + ".down"));
+            float* base = gu.data() + (size_t)e * first_rows * hidden_;
+            std::vector<float> g;
+            if (gated_) g = host_floats(need_tensor(file, ep + ".gate"));
+            else std::memcpy(base, u.data(), u.size() * 4);
+            for (int f = 0; gated_ && f < ff_; ++f) {
                 std::memcpy(base + (size_t)(2 * f) * hidden_, &g[(size_t)f * hidden_], (size_t)hidden_ * 4);
                 std::memcpy(base + (size_t)(2 * f + 1) * hidden_, &u[(size_t)f * hidden_], (size_t)hidden_ * 4);
             }
@@ -325,9 +352,11 @@ public:
             if (shared_gated_) shared_gate_ = f32(".shared.sg");
         }
     }
+    // rows of an expert's first product: two a hidden unit with a gate, else one
+    int first_product_rows() const { return gated_ ? 2 * ff_ : ff_; }
     // a step reads the router, and per token `top` experts at most (all of them once there are many tokens)
     size_t weight_bytes() const override {
-        return (size_t)(experts_ + identity_) * hidden_ * 4 + (size_t)std::min(top_, experts_) * 3 * ff_ * hidden_ * dtype_size(dtype_) +
+        return (size_t)(experts_ + identity_) * hidden_ * 4 + (size_t)std::min(top_, experts_) * (gated_ ? 3 : 2) * ff_ * hidden_ * dtype_size(dtype_) +
                (shared_ ? shared_->weight_bytes() + (size_t)hidden_ * 4 : 0);
     }
     size_t arena_bytes(long long T) const override {
@@ -348,7 +377,8 @@ public:
         float* gate = gated ? ctx.take<float>((size_t)T) : nullptr;
         float* scores = ctx.take<float>((size_t)T * (experts_ + identity_));
         launch_check(eg_moe_route(ctx.stream, (int)dtype, h.p, h.ld, router_.as<float>(), corrected_ ? correction_.as<float>() : nullptr,
-                                  gated ? shared_gate_.as<float>() : nullptr, scores, ids, weights, gate, T, hidden_, experts_ + identity_, top_, sigmoid_ ? 1 : 0),
+                                  gated ? shared_gate_.as<float>() : nullptr, scores, ids, weights, gate, T, hidden_, experts_ + identity_, top_, sigmoid_ ? 1 : 0,
+                                  groups_, keep_groups_, normalize_ ? 1 : 0),
                      "moe_route");
         // where the weight multiplies an expert's input, the sums over the chosen experts count every term once
         const float* in_w = weight_input_ ? weights : nullptr;
@@ -360,7 +390,7 @@ public:
             shared = shared_->forward(ctx, rows, nullptr);
         }
         float* out = ctx.take<float>((size_t)T * hidden_);
-        if (plans::moe_grouped_takes(dtype, T, hidden_, ff_, experts_)) {
+        if (plans::moe_grouped_takes(dtype, T, hidden_, ff_, experts_, gated_)) {
             // many tokens: rows sorted by expert, one grouped product on the tensor cores per projection
             const int max_rows = grouped_rows(T);
             int* scratch = ctx.take<int>((size_t)3 * experts_ + 1 + max_rows / 128 + (size_t)T * top_);
@@ -374,8 +404,8 @@ public:
                 launch_check(eg_gemm_tcgen05_grouped_glu(ctx.stream, rows, hidden_, gate_up_.get(), hidden_, hidden, ff_, max_rows, 2 * ff_, hidden_, experts_,
                                                          tile_group, ctx.status, limit_), "gemm_tcgen05_grouped_glu");
             else
-                launch_check(eg_gemm_tcgen05_grouped(ctx.stream, plans::EPI_SWIGLU, rows, hidden_, gate_up_.get(), hidden_, hidden, ff_, max_rows, 2 * ff_, hidden_,
-                                                     experts_, tile_group, ctx.status), "gemm_tcgen05_grouped");
+                launch_check(eg_gemm_tcgen05_grouped(ctx.stream, gated_ ? plans::EPI_SWIGLU : plans::EPI_GELU, rows, hidden_, gate_up_.get(), hidden_, hidden, ff_,
+                                                     max_rows, first_product_rows(), hidden_, experts_, tile_group, ctx.status), "gemm_tcgen05_grouped");
             launch_check(eg_gemm_tcgen05_grouped(ctx.stream, plans::EPI_STORE, hidden, ff_, down_.get(), ff_, rows, hidden_, max_rows, hidden_, ff_, experts_,
                                                  tile_group, ctx.status), "gemm_tcgen05_grouped");
             launch_check(eg_moe_gather(ctx.stream, rows, row_of, ids, out_w, h.p, h.ld, shared.p, (int)shared.dtype, gate, out, T, hidden_, top_, experts_),
@@ -386,7 +416,8 @@ public:
             return d;
         }
         void* act = ctx.take_rows((size_t)T * top_, std::max(ff_, 1), dtype);
-        launch_check(eg_moe_hidden(ctx.stream, (int)dtype, h.p, h.ld, gate_up_.get(), ids, in_w, act, T, hidden_, ff_, top_, experts_, clamped_ ? 1 : 0, limit_),
+        launch_check(eg_moe_hidden(ctx.stream, (int)dtype, h.p, h.ld, gate_up_.get(), ids, in_w, act, T, hidden_, ff_, top_, experts_, clamped_ ? 1 : gated_ ? 0 : 2,
+                                   limit_),
                      "moe_hidden");
         launch_check(eg_moe_combine(ctx.stream, (int)dtype, h.p, h.ld, act, down_.get(), ids, out_w, shared.p, (int)shared.dtype, gate, out, T, hidden_, ff_,
                                     top_, experts_), "moe_combine");
@@ -398,10 +429,12 @@ public:
 
 private:
     int hidden_, experts_, identity_, top_, ff_, shared_ff_;
-    bool sigmoid_, corrected_, clamped_, weight_input_, shared_gated_;
+    bool sigmoid_, corrected_, clamped_, weight_input_, shared_gated_, gated_;
+    int groups_, keep_groups_;
+    bool normalize_;
     float limit_;
     DType dtype_ = DType::BF16;
-    std::shared_ptr<SwiGLU> shared_;
+    std::shared_ptr<FeedForward> shared_;
     DeviceBuffer router_, correction_, gate_up_, down_, shared_gate_;
 };
 

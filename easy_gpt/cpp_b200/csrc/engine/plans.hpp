@@ -30,7 +30,7 @@ inline int use_pdl() {
     }
     return mode;
 }
-enum Epilogue { EPI_STORE = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_QKV_ROPE = 3, EPI_RESID_NORM = 4, EPI_XIELU = 5 };
+enum Epilogue { EPI_STORE = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_QKV_ROPE = 3, EPI_RESID_NORM = 4, EPI_XIELU = 5, EPI_GELU = 7 };
 
 inline int sm_count() {
     static int count = 0;
@@ -166,10 +166,11 @@ inline int latent_attention_splits(int tokens, int heads, long long max_context)
 
 // Routed experts: from how many tokens on a step's rows are sorted by expert for one grouped product per projection on
 // the tensor cores, instead of every token reading its experts' weights itself.  The grouped product takes widths that
-// are multiples of 128 and expert sizes that are multiples of 64.
+// are multiples of 128 and expert sizes that are multiples of 64 (of 128 without a gate: then a row of the first product's weights is
+// a hidden unit, with a gate two are).
 constexpr int MOE_GROUPED_MIN_TOKENS = 33;
-inline bool moe_grouped_takes(DType dtype, int tokens, int width, int ff, int experts) {
-    return dtype == DType::BF16 && tokens >= MOE_GROUPED_MIN_TOKENS && experts > 0 && width % 128 == 0 && ff % 64 == 0 && ff > 0;
+inline bool moe_grouped_takes(DType dtype, int tokens, int width, int ff, int experts, bool gated = true) {
+    return dtype == DType::BF16 && tokens >= MOE_GROUPED_MIN_TOKENS && experts > 0 && width % 128 == 0 && ff % (gated ? 64 : 128) == 0 && ff > 0;
 }
 
 // How many of a channel's states one thread of the selective scan keeps (1, 2, 4, ... 32): as many as still leave four

@@ -91,7 +91,7 @@ struct Params {
     bf16* xn_out;                //   bfloat16(gain_out * v) [M, N]
     float* ss_out;               //   [gridDim.x][padded tokens]
     // EPI_STORE with an activation on the way out: act 1: act(z) = act_a z^2 + z / 2 for z > 0, act_b (e^z - 1 - z) + z / 2
-    // below; act 2: act(z) = max(z, 0)^2.  EPI_SWIGLU with act 3: g = min(gate, act_a), u = clamp(up, -act_a, act_a),
+    // below; act 2: act(z) = max(z, 0)^2; act 4: the exact gelu.  EPI_SWIGLU with act 3: g = min(gate, act_a), u = clamp(up, -act_a, act_a),
     // out = g sigmoid(1.702 g) (u + 1)
     int act;
     float act_a, act_b;
@@ -506,6 +506,7 @@ __global__ void __launch_bounds__(MAX_THREADS) skinny_kernel(const Params p) {
             float v = value(r, m);
             if (EPI == EPI_STORE && p.act == 1) v = v > 0.f ? fmaf(p.act_a * v, v, 0.5f * v) : fmaf(p.act_b, expm1f(v) - v, 0.5f * v);
             if (EPI == EPI_STORE && p.act == 2) v = v > 0.f ? v * v : 0.f;
+            if (EPI == EPI_STORE && p.act == 4) v = gelu_erf(v);
             if (EPI == EPI_F32) p.out_f32[(size_t)m * p.ldo + n] = v;
             else p.out[(size_t)m * p.ldo + n] = __float2bfloat16_rn(v);
         }
@@ -768,6 +769,16 @@ EG_API int eg_gemm_skinny_relu2(cudaStream_t stream, int use_pdl, const void* W,
     return gemm_skinny_any(stream, EPI_STORE, 0, use_pdl, W, ldw, nullptr, M, N, K, x, ldx, nullptr, nullptr, nullptr, nullptr, 0.f, out, ldo, row_blocks,
                            k_slices, k_split, scratch, counters, 0, 0, 0, nullptr, nullptr, nullptr, nullptr, nullptr, 0, 0, 0, 0, status, nullptr, 0,
                            nullptr, nullptr, 0, nullptr, nullptr, nullptr, nullptr, 2, 0.f, 0.f);
+}
+
+// out [M, N] bfloat16 = gelu(x W^T) (the exact one, by erf), applied to the finished sums.  Sizes, plan and scratch as eg_gemm_skinny with
+// a plain store; with norm 1 or 2 the input is a norm as in eg_gemm_skinny (x null).
+EG_API int eg_gemm_skinny_gelu(cudaStream_t stream, int norm, int use_pdl, const void* W, long long ldw, int M, int N, int K, const void* x, long long ldx,
+                               const float* resid_in, float* resid_out, const void* delta, const float* gain, float eps, const float* ss_in, int ss_parts, void* out,
+                               long long ldo, int row_blocks, int k_slices, int k_split, float* scratch, int* counters, int* status) {
+    return gemm_skinny_any(stream, EPI_STORE, norm, use_pdl, W, ldw, nullptr, M, N, K, x, ldx, resid_in, resid_out, delta, gain, eps, out, ldo, row_blocks,
+                           k_slices, k_split, scratch, counters, 0, 0, 0, nullptr, nullptr, nullptr, nullptr, nullptr, 0, 0, 0, 0, status, nullptr, 0,
+                           nullptr, ss_in, ss_parts, nullptr, nullptr, nullptr, nullptr, 4, 0.f, 0.f);
 }
 
 // out [M, N / 2] bfloat16 from interleaved rows of W (2i = gate_i, 2i + 1 = up_i) with the clamped gate on the finished sums:

@@ -43,7 +43,7 @@ constexpr int THREADS = 192;                                     // 6 warps
 constexpr int TMEM_COLS = 128;
 constexpr unsigned WAIT_LIMIT = 1u << 24;
 
-enum { EPI_STORE = 0, EPI_SWIGLU = 2, EPI_XIELU = 5, EPI_RELU2 = 6 };
+enum { EPI_STORE = 0, EPI_SWIGLU = 2, EPI_XIELU = 5, EPI_RELU2 = 6, EPI_GELU = 7 };
 
 
 // Bounded wait: false if it gave up (or another role already did).
@@ -138,7 +138,8 @@ struct Params {
     const int* tile_group;
     // EPI_XIELU (pair kernel): out = a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 for z <= 0, element by element
     float act_a = 0.f, act_b = 0.f;
-    // EPI_SWIGLU with glu_limit > 0: the clamped gate (glu_fast).  EPI_RELU2 (pair kernel): out = max(z, 0)^2
+    // EPI_SWIGLU with glu_limit > 0: the clamped gate (glu_fast).  EPI_RELU2 (pair kernel): out = max(z, 0)^2.
+    // EPI_GELU (pair and grouped kernels): out = z / 2 (1 + erf(z / sqrt 2))
     float glu_limit = 0.f;
 };
 
@@ -254,6 +255,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         dst[0] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
                         dst[1] = make_uint4(packed[4], packed[5], packed[6], packed[7]);
                     } else {
+                        if (p.epilogue == EPI_GELU) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) v[j] = gelu_erf(v[j]);
+                        }
                         uint32_t packed[16];
 #pragma unroll
                         for (int j = 0; j < 16; ++j) {
@@ -677,6 +682,10 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
 #pragma unroll
                             for (int j = 0; j < 32; ++j) v[j] = v[j] > 0.f ? v[j] * v[j] : 0.f;
                         }
+                        if (p.epilogue == EPI_GELU) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) v[j] = gelu_erf(v[j]);
+                        }
                         uint32_t packed[16];
 #pragma unroll
                         for (int j = 0; j < 16; ++j) {
@@ -1011,7 +1020,7 @@ static int gemm_tcgen05_grouped_any(cudaStream_t stream, int epilogue, const voi
                                    long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, int* status, float glu_limit) {
     if (max_rows <= 0 || N <= 0 || groups <= 0) return 0;
     if (max_rows % BM || N % BN || K % BK || K <= 0 || lda % 8 || ldw % 8 || ldo % 8 || (uintptr_t)A % 16 || (uintptr_t)W % 16 || (uintptr_t)out % 16 ||
-        (epilogue != EPI_STORE && epilogue != EPI_SWIGLU) || !status || !tile_group)
+        (epilogue != EPI_STORE && epilogue != EPI_SWIGLU && epilogue != EPI_GELU) || !status || !tile_group)
         return (int)cudaErrorInvalidValue;
     CUtensorMap map_a, map_w;
     if (make_map(&map_a, A, max_rows, K, lda, BM) || make_map(&map_w, W, (long long)groups * N, K, ldw, BN)) return (int)cudaErrorInvalidValue;
@@ -1028,6 +1037,7 @@ static int gemm_tcgen05_grouped_any(cudaStream_t stream, int epilogue, const voi
     return eg_launch_status();
 }
 
+// epilogue: 0 store, 2 SwiGLU on interleaved columns, 7 the exact gelu (by erf).
 EG_API int eg_gemm_tcgen05_grouped(cudaStream_t stream, int epilogue, const void* A, long long lda, const void* W, long long ldw, void* out,
                                    long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, int* status) {
     return gemm_tcgen05_grouped_any(stream, epilogue, A, lda, W, ldw, out, ldo, max_rows, N, K, groups, tile_group, status, 0.f);
@@ -1111,7 +1121,8 @@ static int gemm_tcgen05_pair_any(cudaStream_t stream, int epilogue, const void* 
                                  long long* trace, float act_a, float act_b) {
     if (M <= 0 || N <= 0) return 0;
     if ((tile_n != 128 && tile_n != 256) || N % tile_n || K % BK || K <= 0 || lda % 8 || ldw % 8 || ldo % 8 || (uintptr_t)A % 16 ||
-        (uintptr_t)W % 16 || (uintptr_t)out % 16 || (epilogue != EPI_STORE && epilogue != EPI_SWIGLU && epilogue != EPI_XIELU && epilogue != EPI_RELU2) ||
+        (uintptr_t)W % 16 || (uintptr_t)out % 16 || (epilogue != EPI_STORE && epilogue != EPI_SWIGLU && epilogue != EPI_XIELU && epilogue != EPI_RELU2 &&
+                                  epilogue != EPI_GELU) ||
         (epilogue == EPI_SWIGLU && tile_n != 256) || !status)
         return (int)cudaErrorInvalidValue;
     static int sm_count = 0;
@@ -1134,7 +1145,7 @@ static int gemm_tcgen05_pair_any(cudaStream_t stream, int epilogue, const void* 
 EG_API int eg_gemm_tcgen05_pair(cudaStream_t stream, int epilogue, const void* A, long long lda, const void* W, long long ldw,
                                 const float* bias, void* out, long long ldo, int M, int N, int K, int tile_n, int* status,
                                 long long* trace) {
-    if (epilogue == EPI_XIELU || epilogue == EPI_RELU2) return (int)cudaErrorInvalidValue;
+    if (epilogue == EPI_XIELU || epilogue == EPI_RELU2 || epilogue == EPI_GELU) return (int)cudaErrorInvalidValue;
     return gemm_tcgen05_pair_any(stream, epilogue, A, lda, W, ldw, bias, out, ldo, M, N, K, tile_n, status, trace, 0.f, 0.f);
 }
 
@@ -1149,6 +1160,12 @@ EG_API int eg_gemm_tcgen05_pair_xielu(cudaStream_t stream, const void* A, long l
 EG_API int eg_gemm_tcgen05_pair_relu2(cudaStream_t stream, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int M,
                                       int N, int K, int tile_n, int* status) {
     return gemm_tcgen05_pair_any(stream, EPI_RELU2, A, lda, W, ldw, nullptr, out, ldo, M, N, K, tile_n, status, nullptr, 0.f, 0.f);
+}
+
+// The same product with the exact gelu in its epilogue: out = z / 2 (1 + erf(z / sqrt 2)), z = A W^T, bfloat16 [M, N].
+EG_API int eg_gemm_tcgen05_pair_gelu(cudaStream_t stream, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int M,
+                                     int N, int K, int tile_n, int* status) {
+    return gemm_tcgen05_pair_any(stream, EPI_GELU, A, lda, W, ldw, nullptr, out, ldo, M, N, K, tile_n, status, nullptr, 0.f, 0.f);
 }
 
 // The same product over interleaved gate and up columns with the clamped gate in its epilogue, out bfloat16 [M, N / 2]:

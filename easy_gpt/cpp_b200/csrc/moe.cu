@@ -18,7 +18,9 @@
 // The sizes of the runs stay on the device: nothing here waits for the host.
 // Products accumulate in float32; the router is float32 throughout.
 //
-// Variants, each a parameter: `scoring` 1 takes s = sigmoid(logits) instead of the softmax (the correction may then be null);
+// Variants, each a parameter: `groups` > 1 cuts the outputs into that many equal runs of neighbours, a group counting the sum of its
+// two largest s + correction, and only outputs of the `keep` best groups can be chosen (ties: the lower group); `normalize` divides
+// a token's weights by their sum (+ 1e-20); `activation` 2 is an expert without a gate, a = gelu(U_e h) (then GU [experts, ff, width]); `scoring` 1 takes s = sigmoid(logits) instead of the softmax (the correction may then be null);
 // `activation` 1 is the clamped gate g' = min(g, limit), u' = clamp(u, -limit, limit), a = g' sigmoid(1.702 g') (u' + 1);
 // `input_weights` (eg_moe_hidden, eg_moe_dispatch) multiply an expert's INPUT row, expert(w h), and eg_moe_combine / eg_moe_gather
 // then get null weights (every term counts once); a null gate adds the shared expert's output as it is.
@@ -47,9 +49,12 @@ __global__ void __launch_bounds__(256) moe_logits_kernel(const T* __restrict__ h
     }
 }
 
-// a warp per token: softmax over the logits (left in place as scores), then the `top` largest of score + correction
+// a warp per token: softmax over the logits (left in place as scores), then the `top` largest of score + correction, within the
+// `keep` best groups; shared memory: `groups` floats per warp (with groups > 1)
 __global__ void __launch_bounds__(128) moe_select_kernel(float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ ids,
-                                                         float* __restrict__ weights, int tokens, int outputs, int top, int scoring) {
+                                                         float* __restrict__ weights, int tokens, int outputs, int top, int scoring, int groups, int keep,
+                                                         int normalize) {
+    extern __shared__ float group_scores[];
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (t >= tokens) return;
     float* logit = logits + (size_t)t * outputs;
@@ -65,12 +70,38 @@ __global__ void __launch_bounds__(128) moe_select_kernel(float* __restrict__ log
         for (int e = lane; e < outputs; e += 32) logit[e] = expf(logit[e] - top_logit) / sum;      // now the scores s
     }
     __syncwarp();
+    const int per = outputs / groups;
+    float* group = group_scores + (size_t)(threadIdx.x >> 5) * groups;
+    if (groups > 1) {
+        for (int g = lane; g < groups; g += 32) {
+            float first = -INFINITY, second = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                const float v = logit[e] + (correction ? correction[e] : 0.f);
+                if (v > first) { second = first; first = v; }
+                else if (v > second) second = v;
+            }
+            group[g] = per > 1 ? first + second : first;
+        }
+        __syncwarp();
+        unsigned long long kept = 0ull;          // bit i for the lane's group lane + 32 i: fewer than `keep` groups come before it
+        for (int g = lane, i = 0; g < groups; g += 32, ++i) {
+            const float mine = group[g];
+            int before = 0;
+            for (int o = 0; o < groups; ++o) before += group[o] > mine || (group[o] == mine && o < g);
+            if (before < keep) kept |= 1ull << i;
+        }
+        __syncwarp();
+        for (int g = lane, i = 0; g < groups; g += 32, ++i) group[g] = (kept >> i) & 1ull ? 1.f : 0.f;
+        __syncwarp();
+    }
+    float sum_chosen = 0.f;
     unsigned long long taken = 0ull;             // a lane tracks which of its own outputs are taken: bit k for e = lane + 32 k
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int arg = 0x7fffffff;
         for (int e = lane, i = 0; e < outputs; e += 32, ++i) {
             if ((taken >> i) & 1ull) continue;
+            if (groups > 1 && group[e / per] == 0.f) continue;
             const float v = logit[e] + (correction ? correction[e] : 0.f);
             if (v > best) { best = v; arg = e; }
         }
@@ -81,15 +112,19 @@ __global__ void __launch_bounds__(128) moe_select_kernel(float* __restrict__ log
         }
         if (arg != 0x7fffffff && arg % 32 == lane) taken |= 1ull << (arg / 32);
         if (lane == 0) {
+            const float s = arg == 0x7fffffff ? 0.f : logit[arg];
             ids[(size_t)t * top + k] = arg == 0x7fffffff ? outputs : arg;
-            weights[(size_t)t * top + k] = arg == 0x7fffffff ? 0.f : logit[arg];
+            weights[(size_t)t * top + k] = s;
+            sum_chosen += s;
         }
     }
+    if (normalize && lane == 0)
+        for (int k = 0; k < top; ++k) weights[(size_t)t * top + k] /= sum_chosen + 1e-20f;
 }
 
 // grid (token, choice, chunk of ff); a warp per hidden unit; GU [experts, 2 ff, width] with the gate row of unit f at
-// 2 f and its up row at 2 f + 1
-template <typename T>
+// 2 f and its up row at 2 f + 1, or without a gate (GATED false) [experts, ff, width]
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(256) moe_hidden_kernel(const T* __restrict__ h, long long ld, const T* __restrict__ GU, const int* __restrict__ ids,
                                                          const float* __restrict__ input_weights, T* __restrict__ act, int width, int ff, int top,
                                                          int experts, int activation, float limit) {
@@ -102,15 +137,15 @@ __global__ void __launch_bounds__(256) moe_hidden_kernel(const T* __restrict__ h
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int f = blockIdx.z * warps + warp;
     if (f >= ff) return;
-    const T* g = GU + ((size_t)e * 2 * ff + 2 * f) * width;
-    const T* u = g + width;
+    const T* g = GU + (GATED ? (size_t)e * 2 * ff + 2 * f : (size_t)e * ff + f) * width;
+    const T* u = GATED ? g + width : g;
     float ag = 0.f, au = 0.f;
     if (sizeof(T) == 2 && width % 8 == 0) {                      // eight weights a load
         const uint4* g8 = reinterpret_cast<const uint4*>(g);
         const uint4* u8 = reinterpret_cast<const uint4*>(u);
 #pragma unroll 2
         for (int j = lane; j < width / 8; j += 32) {
-            const uint4 gv = g8[j], uv = u8[j];
+            const uint4 gv = g8[j], uv = GATED ? u8[j] : gv;
             const __nv_bfloat162* gp = reinterpret_cast<const __nv_bfloat162*>(&gv);
             const __nv_bfloat162* up = reinterpret_cast<const __nv_bfloat162*>(&uv);
 #pragma unroll
@@ -118,25 +153,29 @@ __global__ void __launch_bounds__(256) moe_hidden_kernel(const T* __restrict__ h
                 const float2 gf = __bfloat1622float2(gp[q]), uf = __bfloat1622float2(up[q]);
                 ag = fmaf(gf.x, row[8 * j + 2 * q], ag);
                 ag = fmaf(gf.y, row[8 * j + 2 * q + 1], ag);
-                au = fmaf(uf.x, row[8 * j + 2 * q], au);
-                au = fmaf(uf.y, row[8 * j + 2 * q + 1], au);
+                if (GATED) {
+                    au = fmaf(uf.x, row[8 * j + 2 * q], au);
+                    au = fmaf(uf.y, row[8 * j + 2 * q + 1], au);
+                }
             }
         }
     } else {
         for (int j = lane; j < width; j += 32) {
             ag = fmaf(to_f32<T>(g[j]), row[j], ag);
-            au = fmaf(to_f32<T>(u[j]), row[j], au);
+            if (GATED) au = fmaf(to_f32<T>(u[j]), row[j], au);
         }
     }
     ag = warp_sum(ag);
-    au = warp_sum(au);
+    if (GATED) au = warp_sum(au);
     if (input_weights) {                                         // the expert reads w h: its two products are w times these
         const float wgt = input_weights[(size_t)t * top + k];
         ag *= wgt;
         au *= wgt;
     }
     float a;
-    if (activation == 1) {
+    if (!GATED) {
+        a = gelu_erf(ag);
+    } else if (activation == 1) {
         ag = fminf(ag, limit);
         au = fminf(fmaxf(au, -limit), limit);
         a = ag / (1.0f + expf(-1.702f * ag)) * (au + 1.0f);
@@ -199,13 +238,16 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const T* __restrict__ 
 // ids [T, top] int32 (router outputs; those >= the number of experts stand for the identity), weights [T, top] float32,
 // gate [T] float32 (only with gate_w); logits [T, outputs] float32 is scratch (it ends up holding the scores)
 EG_API int eg_moe_route(cudaStream_t stream, int dtype, const void* h, long long ld, const float* router, const float* correction, const float* gate_w,
-                        float* logits, int* ids, float* weights, float* gate, int tokens, int width, int outputs, int top, int scoring) {
+                        float* logits, int* ids, float* weights, float* gate, int tokens, int width, int outputs, int top, int scoring, int groups, int keep,
+                        int normalize) {
     if (tokens <= 0) return 0;
+    if (groups < 1 || outputs % groups || keep < 1 || keep > groups) return (int)cudaErrorInvalidValue;
     if (top < 1 || top > outputs || outputs > 2048 || !logits || scoring < 0 || scoring > 1) return (int)cudaErrorInvalidValue;
     dim3 grid(tokens, (outputs + (gate_w ? 1 : 0) + 7) / 8);
     if (dtype == EG_BF16) moe_logits_kernel<bf16><<<grid, 256, 0, stream>>>((const bf16*)h, ld, router, gate_w, logits, gate, width, outputs);
     else moe_logits_kernel<float><<<grid, 256, 0, stream>>>((const float*)h, ld, router, gate_w, logits, gate, width, outputs);
-    moe_select_kernel<<<(tokens + 3) / 4, 128, 0, stream>>>(logits, correction, ids, weights, tokens, outputs, top, scoring);
+    const size_t smem = groups > 1 ? (size_t)4 * groups * sizeof(float) : 0;
+    moe_select_kernel<<<(tokens + 3) / 4, 128, smem, stream>>>(logits, correction, ids, weights, tokens, outputs, top, scoring, groups, keep, normalize);
     return eg_launch_status();
 }
 
@@ -216,8 +258,10 @@ EG_API int eg_moe_hidden(cudaStream_t stream, int dtype, const void* h, long lon
     const size_t smem = (size_t)width * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     dim3 grid(tokens, top, (ff + 7) / 8);
-    if (dtype == EG_BF16) moe_hidden_kernel<bf16><<<grid, 256, smem, stream>>>((const bf16*)h, ld, (const bf16*)gate_up, ids, input_weights, (bf16*)act, width, ff, top, experts, activation, limit);
-    else moe_hidden_kernel<float><<<grid, 256, smem, stream>>>((const float*)h, ld, (const float*)gate_up, ids, input_weights, (float*)act, width, ff, top, experts, activation, limit);
+#define EG_HIDDEN(T, G) moe_hidden_kernel<T, G><<<grid, 256, smem, stream>>>((const T*)h, ld, (const T*)gate_up, ids, input_weights, (T*)act, width, ff, top, experts, activation, limit)
+    if (dtype == EG_BF16) { if (activation == 2) EG_HIDDEN(bf16, false); else EG_HIDDEN(bf16, true); }
+    else { if (activation == 2) EG_HIDDEN(float, false); else EG_HIDDEN(float, true); }
+#undef EG_HIDDEN
     return eg_launch_status();
 }
 
