@@ -32,6 +32,7 @@ For profiling and for further sizes (one short line each, never the JSON line ab
     python bench.py --only lasizen [--batch B] [--context C] [--steps K] [--sizes small|medium]
     python bench.py --only mozalix [--batch B] [--context C] [--steps K] [--sizes small|medium] [--model both|mozalix|lasizen]
     python bench.py --only zodosun [--batch B] [--context C] [--steps K] [--sizes small|medium] [--model both|zodosun|mozalix]
+    python bench.py --only mipurax [--batch B] [--context C] [--steps K] [--sizes small|medium] [--model both|mipurax|gufanex]
 
 `gufanex` measures the Gufanex decoder (selective-scan and latent-attention layers with routed experts) at layer sizes
 of real models of those kinds, with random weights, beside a Qwen2 decoder of the same width, depth and active
@@ -48,6 +49,10 @@ biases) the same way, beside the Lasizen decoder of the same width, layer runs a
 `zodosun` measures the Zodosun decoder (attention with sigmoid weights and a bias by distance beside a linear attention with a
 fading state, delta-rule mixers with a decay and a removal rate per key channel, norms in groups) the same way, beside the
 Mozalix decoder of the same width, layer runs and feed-forward.
+
+`mipurax` measures the Mipurax decoder (latent attention with an output gate, attention in chunks with a slope by distance and a
+layer that reads another layer's keys, exact-gelu experts chosen within groups) the same way, beside a Gufanex decoder of latent
+attention and routed experts of the same width, layers, latent sizes and active weights.
 
 `serve` runs 64 concurrent requests (prompts of 128..4096 tokens in portions of 512 beside
 decoding requests, 512 new tokens each) through the engine and reports wall-clock tokens a second.
@@ -183,6 +188,28 @@ def zodosun_bench_configs(size):
     zodosun = {"architecture": "Zodosun", "vocab": 32000, "width": width, "norm": {"eps": 1e-6, "groups": 4}, "logit_scale": 0.5,
                "layers": [dict(m, mlp=mlp) for m in (delta, pair, delta, delta, pair, delta)]}
     return zodosun, mozalix_bench_configs(size)[0]
+
+
+# Layer sizes for `--only mipurax`: width 2,048; latent attention of 16 heads (128 plain and 64 turned query/key values, values of 128,
+# latents of 512 and 1,536) in both forms; an attention of 16 heads of 128 over 4 key heads in chunks of 1,024, a second one reading its
+# keys; 64 experts of 1,536 in 8 groups (4 kept), six a token, beside a shared one of 3,072, or a dense feed-forward of as many active
+# weights ("medium"); half of the width, heads, experts and feed-forwards ("small").  Six layers.  Beside it the closest existing
+# model: six Gufanex layers of latent attention of the same sizes with gated experts of 1,024 (as many weights an expert).
+def mipurax_bench_configs(size):
+    k = {"medium": 1, "small": 2}[size]
+    width, ff, heads = 2048 // k, 1536 // k, 16 // k
+    sizes = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 1536 // k, "scale": 192 ** -0.5,
+             "rot": {"base": 10000.0, "dims": 64}}
+    first, second = {"type": "latent_attention", "mixer": sizes}, {"type": "latent_attention_2", "mixer": sizes}
+    chunked = {"type": "attention", "mixer": {"heads": heads, "kv_heads": 4 // k, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024}}}
+    moe = {"kind": "moe", "router": {"experts": 64 // k, "top": 6, "groups": {"count": 8, "keep": 4}}, "expert": {"ff": ff}, "shared": {"ff": 2 * ff}}
+    dense = {"kind": "dense", "ff": 8 * ff}
+    reader = {"type": "attention", "mixer": dict(chunked["mixer"], kv_from=1)}
+    mipurax = {"architecture": "Mipurax", "vocab": 32000, "width": width, "norm": {"eps": 1e-6},
+               "layers": [dict(first, mlp=dense), dict(chunked, mlp=moe), dict(second, mlp=moe), dict(first, mlp=moe), dict(reader, mlp=dense), dict(second, mlp=moe)]}
+    gated = {"kind": "moe", "expert": {"ff": 2 * ff // 3}, "router": {"experts": 64 // k, "identity": 0, "top": 6}, "shared": {"ff": 4 * ff // 3}}
+    gufanex = {"architecture": "Gufanex", "vocab": 32000, "width": width, "norm": {"eps": 1e-6}, "layers": [dict(first, mlp=gated)] * 6}
+    return mipurax, gufanex
 
 
 CONTEXT = 4096
@@ -374,6 +401,8 @@ def gufanex_folder(config, seed=0):
         from easy_gpt.cpp_b200.weights.mozalix_init import write_random_model
     elif config.get("architecture") == "Zodosun":
         from easy_gpt.cpp_b200.weights.zodosun_init import write_random_model
+    elif config.get("architecture") == "Mipurax":
+        from easy_gpt.cpp_b200.weights.mipurax_init import write_random_model
     else:
         from easy_gpt.cpp_b200.weights.gufanex_init import write_random_model
 
@@ -752,7 +781,25 @@ def run_zodosun(args):
     return 0
 
 
+def run_mipurax(args):
+    size = args.sizes if args.sizes in ("small", "medium") else "medium"
+    mipurax, gufanex = mipurax_bench_configs(size)
+    context = min(args.context, 2048) if args.context == CONTEXT else args.context
+    out = {"only": "mipurax", "sizes": size, "batch": args.batch, "context": context, "prefill_tokens": PREFILL_TOKENS, "dtype": "bfloat16",
+           "data": "synthetic (random weights)"}
+    with ClockSampler() as clocks:
+        if args.model in ("both", "mipurax"):
+            out["mipurax"] = measure_prefill_and_decode(gufanex_folder(mipurax), mipurax["vocab"], args.batch, context, args.steps, args.warmup)
+        if args.model in ("both", "gufanex"):
+            out["gufanex_equal"] = measure_prefill_and_decode(gufanex_folder(gufanex), gufanex["vocab"], args.batch, context, args.steps, args.warmup)
+    out["clocks"] = clocks.summary()
+    print(json.dumps(out))
+    return 0
+
+
 def run_ours(args):
+    if args.only == "mipurax":
+        return run_mipurax(args)
     if args.only == "zodosun":
         return run_zodosun(args)
     if args.only == "mozalix":
@@ -890,16 +937,16 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--context", type=int, default=CONTEXT, help="context length the decode steps end at (default 4096)")
-    ap.add_argument("--sizes", choices=list(SIZES) + ["small", "medium"], default="0.5b", help="layer sizes for --only runs (small, medium: --only gufanex, --only lasizen, --only masezen, --only mozalix and --only zodosun)")
-    ap.add_argument("--model", choices=["both", "gufanex", "lasizen", "masezen", "mozalix", "zodosun", "qwen2"], default="both",
-                    help="with --only gufanex, --only lasizen, --only masezen, --only mozalix or --only zodosun: which of the two models to measure")
+    ap.add_argument("--sizes", choices=list(SIZES) + ["small", "medium"], default="0.5b", help="layer sizes for --only runs (small, medium: --only gufanex, --only lasizen, --only masezen, --only mozalix, --only zodosun and --only mipurax)")
+    ap.add_argument("--model", choices=["both", "gufanex", "lasizen", "masezen", "mozalix", "zodosun", "mipurax", "qwen2"], default="both",
+                    help="with --only gufanex, --only lasizen, --only masezen, --only mozalix, --only zodosun or --only mipurax: which of the two models to measure")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16", help="precision of --only decode")
     ap.add_argument("--default-options", action="store_true",
                     help="--only decode with the engine's default page size and request length")
     ap.add_argument("--ref-prompt", type=int, default=0,
                     help="prompt length of the reference arm (0: 1536, or the longest its int-indexed logits allow)")
     ap.add_argument("--fused", action="store_true", help="with --only timeline or decode: the decode step as one persistent kernel (EASY_GPT_FUSED_DECODE=1)")
-    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "gemm", "attention", "serve", "gufanex", "lasizen", "masezen", "mozalix", "zodosun"], default=None,
+    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "gemm", "attention", "serve", "gufanex", "lasizen", "masezen", "mozalix", "zodosun", "mipurax"], default=None,
                     help="measure one part only and print a short line (for profiling runs)")
     args = ap.parse_args()
     if args.gpus != 1:

@@ -248,7 +248,9 @@ def random_weights(config, seed, overrides=None):
             v = 1.0 + 0.2 * rng.standard_normal(shape)
         elif leaf in ("norm1", "norm2", "norm"):
             v = 0.2 * rng.standard_normal(shape)                 # the gain is one plus this
-        elif leaf in ("sink", "embed"):
+        elif leaf == "sink":
+            v = 2.0 + rng.standard_normal(shape)                 # as much as several keys: a sink that is left out shows
+        elif leaf == "embed":
             v = rng.standard_normal(shape)
         else:
             v = rng.standard_normal(shape) * (1.5 / math.sqrt(shape[-1]))
