@@ -25,32 +25,50 @@ __device__ __forceinline__ void store_any(void* p, int dtype, size_t i, float v)
     else ((float*)p)[i] = v;
 }
 
-// one block per token
-__global__ void latent_prepare_kernel(const float* __restrict__ down, long long ld, int q_rank, int rank, int rot, int rot_dims, int rot_half,
-                                      const float* __restrict__ gain_q, const float* __restrict__ gain_c, float eps, const float* __restrict__ inv_freq,
-                                      const int* __restrict__ positions, const int* __restrict__ slot_map, void* __restrict__ cache, int cache_dtype,
-                                      int page_size, long long page_stride, long long pool_slots, void* __restrict__ cq, int cq_dtype,
-                                      int* __restrict__ status) {
+// grid (token, 2): one block norms the query latent, the other the latent and turns the key part.  A thread keeps up to VPT of its row's
+// values in registers (all loads in flight at once); longer rows are read twice.
+constexpr int VPT = 8;
+template <typename Store>
+__device__ __forceinline__ void norm_row(const float* __restrict__ row, int n, const float* __restrict__ gain, float eps, float* scratch, Store store) {
+    float v[VPT], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int j = threadIdx.x + i * blockDim.x;
+        v[i] = j < n ? row[j] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) ss = fmaf(v[i], v[i], ss);
+    for (int j = threadIdx.x + VPT * blockDim.x; j < n; j += blockDim.x) ss = fmaf(row[j], row[j], ss);
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int j = threadIdx.x + i * blockDim.x;
+        if (j < n) store(j, v[i] * inv * gain[j]);
+    }
+    for (int j = threadIdx.x + VPT * blockDim.x; j < n; j += blockDim.x) store(j, row[j] * inv * gain[j]);
+}
+
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const float* __restrict__ down, long long ld, int q_rank, int rank, int rot, int rot_dims, int rot_half,
+                                                             const float* __restrict__ gain_q, const float* __restrict__ gain_c, float eps,
+                                                             const float* __restrict__ inv_freq, const int* __restrict__ positions,
+                                                             const int* __restrict__ slot_map, void* __restrict__ cache, int cache_dtype, int page_size,
+                                                             long long page_stride, long long pool_slots, void* __restrict__ cq, int cq_dtype,
+                                                             int* __restrict__ status) {
     __shared__ float scratch[32];
     const int t = blockIdx.x;
     const float* row = down + (size_t)t * ld;
-    float ss = 0.f;
-    for (int j = threadIdx.x; j < q_rank; j += blockDim.x) ss += row[j] * row[j];
-    const float inv_q = 1.0f / sqrtf(block_sum(ss, scratch) / (float)q_rank + eps);
-    for (int j = threadIdx.x; j < q_rank; j += blockDim.x) store_any(cq, cq_dtype, (size_t)t * q_rank + j, row[j] * inv_q * gain_q[j]);
-    if (!cache) return;
+    if (blockIdx.y == 0) {
+        norm_row(row, q_rank, gain_q, eps, scratch, [&](int j, float v) { store_any(cq, cq_dtype, (size_t)t * q_rank + j, v); });
+        return;
+    }
     const long long slot = slot_map[t];
     if (slot < 0 || slot >= pool_slots) {
         if (threadIdx.x == 0) atomicOr(status, EG_STATUS_BAD_SLOT);
         return;
     }
     const float* c = row + q_rank;
-    ss = 0.f;
-    for (int j = threadIdx.x; j < rank; j += blockDim.x) ss += c[j] * c[j];
-    const float inv_c = 1.0f / sqrtf(block_sum(ss, scratch) / (float)rank + eps);
-    const size_t at = (size_t)(slot / page_size) * page_stride + (size_t)(slot % page_size) * (rank + rot);
-    for (int j = threadIdx.x; j < rank; j += blockDim.x) store_any(cache, cache_dtype, at + j, c[j] * inv_c * gain_c[j]);
     const float* kr = c + rank;
+    const size_t at = (size_t)(slot / page_size) * page_stride + (size_t)(slot % page_size) * (rank + rot);
     const float pos = (float)positions[t];
     for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
         float sn, cs;
@@ -61,6 +79,7 @@ __global__ void latent_prepare_kernel(const float* __restrict__ down, long long 
         store_any(cache, cache_dtype, at + rank + d1, b * cs + a * sn);
     }
     for (int j = rot_dims + threadIdx.x; j < rot; j += blockDim.x) store_any(cache, cache_dtype, at + rank + j, kr[j]);
+    norm_row(c, rank, gain_c, eps, scratch, [&](int j, float v) { store_any(cache, cache_dtype, at + j, v); });
 }
 
 // one block per (token, head); Uk [heads * dim, rank] in TW
@@ -200,7 +219,8 @@ EG_API int eg_latent_prepare(cudaStream_t stream, const float* down, long long l
                              int page_size, long long page_stride, long long pool_slots, void* cq, int cq_dtype, int tokens, int* status) {
     if (tokens <= 0) return 0;
     if (rot_dims % 2 || rot_dims > rot || q_rank <= 0 || rank <= 0) return (int)cudaErrorInvalidValue;
-    latent_prepare_kernel<<<tokens, 128, 0, stream>>>(down, ld, q_rank, rank, rot, rot_dims, rot_half, gain_q, gain_c, eps, inv_freq, positions, slot_map, cache,
+    const dim3 grid(tokens, cache ? 2 : 1);
+    latent_prepare_kernel<<<grid, 256, 0, stream>>>(down, ld, q_rank, rank, rot, rot_dims, rot_half, gain_q, gain_c, eps, inv_freq, positions, slot_map, cache,
                                                      cache_dtype, page_size, page_stride, pool_slots, cq, cq_dtype, status);
     return eg_launch_status();
 }

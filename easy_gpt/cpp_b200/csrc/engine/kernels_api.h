@@ -76,17 +76,25 @@ int eg_moe_hidden(cudaStream_t stream, int dtype, const void* h, long long ld, c
 // moe.cu
 int eg_moe_combine(cudaStream_t stream, int dtype, const void* h, long long ld, const void* act, const void* down, const int* ids, const float* weights, const void* shared, int shared_dtype, const float* gate, float* out, int tokens, int width, int ff, int top, int experts);
 // moe.cu
+int eg_moe_matvec(cudaStream_t stream, int mode, const void* x, long long ldx, int pairs_per_row, const void* W, const int* ids, const float* input_weights, void* out, int pairs, int rows, int K, int experts, int activation, float limit);
+// moe.cu
+int eg_moe_sum(cudaStream_t stream, const float* y, const int* ids, const float* weights, const void* h, long long ld, const void* shared, int shared_dtype, const float* gate, float* out, int tokens, int width, int top, int experts);
+// moe.cu
 int eg_moe_dispatch(cudaStream_t stream, const void* h, long long ld, const int* ids, const float* input_weights, int* counts, int* starts, int* cursors, int* tile_group, int* row_of, void* rows, int tokens, int width, int top, int experts, int max_rows);
 // moe.cu
 int eg_moe_gather(cudaStream_t stream, const void* y, const int* row_of, const int* ids, const float* weights, const void* h, long long ld, const void* shared, int shared_dtype, const float* gate, float* out, int tokens, int width, int top, int experts);
 // gemm_tcgen05.cu
-int eg_gemm_tcgen05_grouped(cudaStream_t stream, int epilogue, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, int* status);
+int eg_gemm_tcgen05_grouped(cudaStream_t stream, int epilogue, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, const int* active_rows, int* status);
 // gemm_tcgen05.cu
 int eg_gemm_tcgen05_few(cudaStream_t stream, int epilogue, int use_pdl, const void* A, long long lda, const void* W, long long ldw, const float* bias, void* out, long long ldo, int M, int N, int K, int tile_n, int slices, float* partial, int* tickets, int* status);
 // attention_latent_mma.cu
 int eg_attention_latent_mma_takes(int rank, int rot);
 // attention_latent_mma.cu
-int eg_attention_latent_mma(cudaStream_t stream, const void* qa, const void* cache, const int* block_table, int table_stride, const int* token_seq, const int* positions, const float* sink, void* out, float* part_o, float* part_ml, int tokens, int heads, int rank, int rot, int page_size, long long page_stride, int num_pages, int splits, int* status);
+int eg_attention_latent_mma(cudaStream_t stream, const void* qa, const void* cache, const int* block_table, int table_stride, const int* token_seq, const int* positions, const int* token_list, const float* sink, void* out, float* part_o, float* part_ml, int tokens, int heads, int rank, int rot, int page_size, long long page_stride, int num_pages, int splits, int* status);
+// attention_latent_mma.cu
+int eg_attention_latent_tiles_tokens(int heads, int rank, int rot);
+// attention_latent_mma.cu
+int eg_attention_latent_tiles(cudaStream_t stream, const void* qa, const void* cache, const int* block_table, int table_stride, const int* tiles, int num_tiles, const int* positions, const float* sink, void* out, float* part_o, float* part_ml, int heads, int rank, int rot, int page_size, long long page_stride, int num_pages, int splits, int tile_stride, int* status);
 // attention_latent_mma.cu
 int eg_latent_rotate_query(cudaStream_t stream, const void* q, long long ldq, const int* positions, const float* inv_freq, int rot_dims, int rot_half, float scale, void* qa, int tokens, int heads, int dim, int rot, int rank);
 // sandwich.cu
@@ -156,7 +164,7 @@ int eg_gemm_tcgen05_pair_relu2(cudaStream_t stream, const void* A, long long lda
 // gemm_tcgen05.cu
 int eg_gemm_tcgen05_pair_glu(cudaStream_t stream, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int M, int N, int K, int* status, float limit);
 // gemm_tcgen05.cu
-int eg_gemm_tcgen05_grouped_glu(cudaStream_t stream, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, int* status, float limit);
+int eg_gemm_tcgen05_grouped_glu(cudaStream_t stream, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, const int* active_rows, int* status, float limit);
 // attention_masked.cu
 int eg_masked_attention_prepare(cudaStream_t stream, int dtype, const float* proj, long long ld, const float* table, int rot_dims, float magnitude, const int* slot_map, void* k_cache, void* v_cache, int row_stride, long long head_stride, int page_size, long long page_stride, long long pool_slots, void* q_out, int tokens, int heads, int kv_heads, int maps, int dk, int dv, float norm_eps, const float* q_gain, const float* k_gain, int planes, int* status);
 // attention_masked.cu

@@ -182,8 +182,8 @@ public:
     size_t arena_bytes(long long T) const override {
         const size_t per_token = (size_t)(q_rank_ + rank_ + rot_ + gates()) * 4 + (size_t)q_rank_ * 4 + (size_t)heads_ * (dim_ + rot_) * 4 + (size_t)heads_ * (rank_ + rot_) * 4 +
                                  (size_t)heads_ * rank_ * 4 + (size_t)heads_ * vdim_ * 4 + (size_t)hidden_ * 4;
-        // the parts of an attention whose keys are cut: at most two CTAs an SM's worth of them beyond one per token
-        const size_t parts = (size_t)(4 * plans::sm_count() + 64) * 16 * (size_t)(rank_ + 2) * 4;
+        // the parts of an attention whose keys are cut: a CTA of 64 rows an SM for prompt portions, two of 16 an SM for single tokens
+        const size_t parts = (size_t)(4 * plans::sm_count() + 64) * 32 * (size_t)(rank_ + 2) * 4;
         return (size_t)T * per_token + parts + (1u << 16);
     }
     bool capturable() const override { return true; }
@@ -221,16 +221,32 @@ public:
                                         (long long)heads_ * D, D, false, heads_);
             launch_check(eg_latent_rotate_query(ctx.stream, q.p, q.ld, ctx.positions, inv_freq_.as<float>(), rot_dims_, rot_half_, scale_, qa, T, heads_, dim_, rot_, rank_),
                          "latent_rotate_query");
-            const int splits = plans::latent_attention_splits(T, heads_, ctx.max_context_len);
-            float *part_o = nullptr, *part_ml = nullptr;
-            if (splits > 1) {
-                part_o = ctx.take<float>((size_t)T * heads_ * splits * rank_);
-                part_ml = ctx.take<float>((size_t)T * heads_ * splits * 2);
-            }
             void* o = ctx.take_rows((size_t)T * heads_, rank_, dtype);
-            launch_check(eg_attention_latent_mma(ctx.stream, qa, cache.k, tables.block_table, tables.table_width, ctx.token_seq, ctx.positions,
-                                                 sink_ ? sinks_.as<float>() : nullptr, o, part_o, part_ml, T, heads_, rank_, rot_, cache.page_size, cache.page_stride,
-                                                 cache.num_pages, splits, ctx.status), "attention_latent_mma");
+            const float* sinks = sink_ ? sinks_.as<float>() : nullptr;
+            float *part_o = nullptr, *part_ml = nullptr;
+            auto take_parts = [&](int splits, size_t places) {
+                if (splits <= 1) return;
+                part_o = ctx.take<float>(places * heads_ * splits * rank_);
+                part_ml = ctx.take<float>(places * heads_ * splits * 2);
+            };
+            // prompt portions: several tokens' heads against a key tile; single tokens and entries of a few: a token's heads
+            const int tile_tokens = ctx.query_tiles ? eg_attention_latent_tiles_tokens(heads_, rank_, rot_) : 0;
+            if (tile_tokens) {
+                const int splits = plans::latent_tiles_splits(ctx.num_tiles, heads_, tile_tokens, ctx.max_query_len, ctx.max_context_len);
+                const int stride = std::min(plans::QUERY_TILE, ctx.max_query_len);
+                take_parts(splits, (size_t)ctx.num_tiles * stride);
+                launch_check(eg_attention_latent_tiles(ctx.stream, qa, cache.k, tables.block_table, tables.table_width, ctx.query_tiles, ctx.num_tiles, ctx.positions,
+                                                       sinks, o, part_o, part_ml, heads_, rank_, rot_, cache.page_size, cache.page_stride, cache.num_pages, splits,
+                                                       stride, ctx.status), "attention_latent_tiles");
+            }
+            const int singles = tile_tokens ? ctx.num_small : T;
+            if (singles > 0) {
+                const int splits = plans::latent_attention_splits(singles, heads_, ctx.max_context_len);
+                take_parts(splits, (size_t)singles);
+                launch_check(eg_attention_latent_mma(ctx.stream, qa, cache.k, tables.block_table, tables.table_width, ctx.token_seq, ctx.positions,
+                                                     tile_tokens ? ctx.small_tokens : nullptr, sinks, o, part_o, part_ml, singles, heads_, rank_, rot_,
+                                                     cache.page_size, cache.page_stride, cache.num_pages, splits, ctx.status), "attention_latent_mma");
+            }
             Rows values{ctx.take_rows(T, heads_ * vdim_, dtype), dtype, T, heads_ * vdim_, heads_ * vdim_};
             ctx.blas->gemm_bf16_batched(ctx.stream, true, vdim_, T, rank_, 1.0f, up_v_.get(), rank_, (long long)vdim_ * rank_, o, (long long)heads_ * rank_, rank_,
                                         values.p, values.ld, vdim_, false, heads_);
@@ -361,7 +377,8 @@ public:
     }
     size_t arena_bytes(long long T) const override {
         const size_t sorted = (size_t)grouped_rows(T) * ((size_t)hidden_ + ff_) * 2 + (size_t)grouped_rows(T) / 32 + (size_t)experts_ * 16;
-        return (size_t)T * ((size_t)top_ * (12 + (size_t)ff_ * 4) + 4 + (size_t)(experts_ + identity_) * 4 + (size_t)hidden_ * 8 + (size_t)shared_ff_ * 3 * 4) + sorted + (1u << 16);
+        return (size_t)T * ((size_t)top_ * (12 + (size_t)ff_ * 4) + 4 + (size_t)(experts_ + identity_) * 4 + (size_t)hidden_ * 8 + (size_t)shared_ff_ * 3 * 4) + sorted +
+               (size_t)std::min<long long>(T, plans::MOE_GROUPED_MIN_TOKENS) * top_ * hidden_ * 4 + (1u << 16);
     }
     // rows of the sorted copy of a step of T tokens: every expert's run starts at a multiple of 128
     int grouped_rows(long long T) const { return (int)((T * top_ + 127) / 128 * 128 + 128LL * experts_); }
@@ -402,12 +419,12 @@ public:
             void* hidden = ctx.take_rows(max_rows, ff_, dtype);
             if (clamped_)
                 launch_check(eg_gemm_tcgen05_grouped_glu(ctx.stream, rows, hidden_, gate_up_.get(), hidden_, hidden, ff_, max_rows, 2 * ff_, hidden_, experts_,
-                                                         tile_group, ctx.status, limit_), "gemm_tcgen05_grouped_glu");
+                                                         tile_group, starts + experts_, ctx.status, limit_), "gemm_tcgen05_grouped_glu");
             else
                 launch_check(eg_gemm_tcgen05_grouped(ctx.stream, gated_ ? plans::EPI_SWIGLU : plans::EPI_GELU, rows, hidden_, gate_up_.get(), hidden_, hidden, ff_,
-                                                     max_rows, first_product_rows(), hidden_, experts_, tile_group, ctx.status), "gemm_tcgen05_grouped");
+                                                     max_rows, first_product_rows(), hidden_, experts_, tile_group, starts + experts_, ctx.status), "gemm_tcgen05_grouped");
             launch_check(eg_gemm_tcgen05_grouped(ctx.stream, plans::EPI_STORE, hidden, ff_, down_.get(), ff_, rows, hidden_, max_rows, hidden_, ff_, experts_,
-                                                 tile_group, ctx.status), "gemm_tcgen05_grouped");
+                                                 tile_group, starts + experts_, ctx.status), "gemm_tcgen05_grouped");
             launch_check(eg_moe_gather(ctx.stream, rows, row_of, ids, out_w, h.p, h.ld, shared.p, (int)shared.dtype, gate, out, T, hidden_, top_, experts_),
                          "moe_gather");
             Delta d;
@@ -416,6 +433,19 @@ public:
             return d;
         }
         void* act = ctx.take_rows((size_t)T * top_, std::max(ff_, 1), dtype);
+        if (plans::moe_matvec_takes(dtype, T, top_, hidden_, ff_, experts_) && h.ld % 8 == 0) {
+            // several tokens: an expert's weights are read once for all that chose it
+            const int pairs = T * top_;
+            launch_check(eg_moe_matvec(ctx.stream, gated_ ? 0 : 1, h.p, h.ld, top_, gate_up_.get(), ids, in_w, act, pairs, first_product_rows(), hidden_, experts_,
+                                       clamped_ ? 1 : 0, limit_), "moe_matvec");
+            float* y = ctx.take<float>((size_t)pairs * hidden_);
+            launch_check(eg_moe_matvec(ctx.stream, 2, act, ff_, 1, down_.get(), ids, nullptr, y, pairs, hidden_, ff_, experts_, 0, 0.f), "moe_matvec");
+            launch_check(eg_moe_sum(ctx.stream, y, ids, out_w, h.p, h.ld, shared.p, (int)shared.dtype, gate, out, T, hidden_, top_, experts_), "moe_sum");
+            Delta d;
+            d.p = out;
+            d.dtype = DType::F32;
+            return d;
+        }
         launch_check(eg_moe_hidden(ctx.stream, (int)dtype, h.p, h.ld, gate_up_.get(), ids, in_w, act, T, hidden_, ff_, top_, experts_, clamped_ ? 1 : gated_ ? 0 : 2,
                                    limit_),
                      "moe_hidden");

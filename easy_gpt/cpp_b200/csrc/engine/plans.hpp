@@ -164,11 +164,24 @@ inline int latent_attention_splits(int tokens, int heads, long long max_context)
     return splits;
 }
 
+// The same for prompt portions in tiles of several tokens, whose CTAs have an SM each.
+inline int latent_tiles_splits(int num_tiles, int heads, int tokens_per_cta, long long longest_portion, long long max_context) {
+    const long long per_tile = (std::min<long long>(128, longest_portion) + tokens_per_cta - 1) / tokens_per_cta;
+    const long long base = num_tiles * per_tile * ((heads + 15) / 16), tiles = std::max<long long>(1, (max_context + 63) / 64);
+    int splits = 1;
+    while ((long long)splits * 2 * base <= sm_count() && splits * 4 <= tiles && splits < 64) splits *= 2;
+    return splits;
+}
+
 // Routed experts: from how many tokens on a step's rows are sorted by expert for one grouped product per projection on
 // the tensor cores, instead of every token reading its experts' weights itself.  The grouped product takes widths that
 // are multiples of 128 and expert sizes that are multiples of 64 (of 128 without a gate: then a row of the first product's weights is
 // a hidden unit, with a gate two are).
 constexpr int MOE_GROUPED_MIN_TOKENS = 33;
+// Between: steps of several tokens whose experts may coincide read an expert's weights once for all of its tokens.
+inline bool moe_matvec_takes(DType dtype, int tokens, int top, int width, int ff, int experts) {
+    return dtype == DType::BF16 && tokens >= 2 && tokens < MOE_GROUPED_MIN_TOKENS && tokens * top <= 512 && experts > 0 && width % 8 == 0 && ff % 8 == 0 && ff > 0;
+}
 inline bool moe_grouped_takes(DType dtype, int tokens, int width, int ff, int experts, bool gated = true) {
     return dtype == DType::BF16 && tokens >= MOE_GROUPED_MIN_TOKENS && experts > 0 && width % 128 == 0 && ff % (gated ? 64 : 128) == 0 && ff > 0;
 }

@@ -133,9 +133,11 @@ struct Params {
     int epilogue;
     int* status;
     long long* trace;          // optional (profiling): clock stamps of the first pair's MMA thread, three per step of K
-    // grouped products (single-CTA kernel only): row tile i of A is multiplied by the W of group tile_group[i] (W holds
-    // the groups' [N, K] matrices one after the other); a tile whose entry is negative has no rows and is skipped
+    // grouped products (single-CTA kernels only): row tile i of A is multiplied by the W of group tile_group[i] (W holds
+    // the groups' [N, K] matrices one after the other); a tile whose entry is negative has no rows and is skipped.  The persistent
+    // kernel takes the number of rows in use from active_rows (a multiple of 128; the tiles behind it are empty)
     const int* tile_group;
+    const int* active_rows = nullptr;
     // EPI_XIELU (pair kernel): out = a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 for z <= 0, element by element
     float act_a = 0.f, act_b = 0.f;
     // EPI_SWIGLU with glu_limit > 0: the clamped gate (glu_fast).  EPI_RELU2 (pair kernel): out = max(z, 0)^2.
@@ -306,7 +308,8 @@ gemm_tcgen05_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
     unsigned char* ring = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int k_blocks = p.K / BK;
-    const int m_tiles = (p.M + BM - 1) / BM, n_tiles = p.N / WBN;
+    const int rows_in_use = p.active_rows ? min(__ldg(p.active_rows), p.M) : p.M;
+    const int m_tiles = (rows_in_use + BM - 1) / BM, n_tiles = p.N / WBN;
     const int total_tiles = m_tiles * n_tiles;
 
     if (threadIdx.x == 0) {
@@ -336,6 +339,7 @@ gemm_tcgen05_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
             bool ok = true;
             for (int t = blockIdx.x; t < total_tiles && ok; t += gridDim.x) {
                 const int n0 = (t / m_tiles) * WBN, m0 = (t % m_tiles) * BM;
+                const int w_row0 = p.tile_group ? max(0, __ldg(p.tile_group + t % m_tiles)) * p.N + n0 : n0;
                 for (int kb = 0; kb < k_blocks; ++kb, ++g) {
                     const int s = g % WSTAGES;
                     if (g >= WSTAGES && !mbar_wait(&empty_bar[s], ((g / WSTAGES) - 1) & 1, &abort_flag, p.status)) { ok = false; break; }
@@ -343,8 +347,8 @@ gemm_tcgen05_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
                     unsigned char* a = ring + s * W_STAGE_BYTES;
                     tma_load_2d(a, &map_a, &full_bar[s], kb * BK, m0);
                     // the W box is 128 rows: two boxes make the 256-row tile
-                    tma_load_2d(a + TILE_A_BYTES, &map_w, &full_bar[s], kb * BK, n0);
-                    tma_load_2d(a + TILE_A_BYTES + TILE_B_BYTES, &map_w, &full_bar[s], kb * BK, n0 + 128);
+                    tma_load_2d(a + TILE_A_BYTES, &map_w, &full_bar[s], kb * BK, w_row0);
+                    tma_load_2d(a + TILE_A_BYTES + TILE_B_BYTES, &map_w, &full_bar[s], kb * BK, w_row0 + 128);
                 }
             }
         }
@@ -425,6 +429,10 @@ gemm_tcgen05_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
                         dst[0] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
                         dst[1] = make_uint4(packed[4], packed[5], packed[6], packed[7]);
                     } else {
+                        if (p.epilogue == EPI_GELU) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) v[j] = gelu_erf(v[j]);
+                        }
                         uint32_t packed[16];
 #pragma unroll
                         for (int j = 0; j < 16; ++j) {
@@ -1015,9 +1023,10 @@ EG_API int eg_gemm_tcgen05(cudaStream_t stream, int epilogue, const void* A, lon
 // Grouped product for routed experts: A [max_rows, K] holds the rows of group after group, each group's rows starting at
 // a multiple of 128; row tile i (128 rows) belongs to group tile_group[i] (device array of max_rows / 128 entries; negative:
 // an empty tile) and is multiplied by that group's W (W [groups * N, K]).  out [max_rows, N] (or [max_rows, N / 2] with the
-// SwiGLU epilogue on interleaved columns), bfloat16.  One launch whatever the groups' sizes, which only the device knows.
+// SwiGLU epilogue on interleaved columns), bfloat16.  One launch whatever the groups' sizes, which only the device knows.  active_rows
+// (a device int, or null): the rows in use, a multiple of 128; with it and N % 256 == 0 the persistent kernel runs.
 static int gemm_tcgen05_grouped_any(cudaStream_t stream, int epilogue, const void* A, long long lda, const void* W, long long ldw, void* out,
-                                   long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, int* status, float glu_limit) {
+                                   long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, const int* active_rows, int* status, float glu_limit) {
     if (max_rows <= 0 || N <= 0 || groups <= 0) return 0;
     if (max_rows % BM || N % BN || K % BK || K <= 0 || lda % 8 || ldw % 8 || ldo % 8 || (uintptr_t)A % 16 || (uintptr_t)W % 16 || (uintptr_t)out % 16 ||
         (epilogue != EPI_STORE && epilogue != EPI_SWIGLU && epilogue != EPI_GELU) || !status || !tile_group)
@@ -1032,6 +1041,22 @@ static int gemm_tcgen05_grouped_any(cudaStream_t stream, int epilogue, const voi
     }
     Params p{(bf16*)out, ldo, nullptr, max_rows, N, K, epilogue, status, nullptr, tile_group};
     p.glu_limit = glu_limit;
+    if (active_rows && N % wide::WBN == 0) {
+        static bool wide_configured = false;
+        static int sm_count = 0;
+        if (!wide_configured) {
+            cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_wide_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, wide::W_SMEM_BYTES);
+            if (e != cudaSuccess) return (int)e;
+            int dev = 0;
+            cudaGetDevice(&dev);
+            if (cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sm_count <= 0) sm_count = 148;
+            wide_configured = true;
+        }
+        p.active_rows = active_rows;
+        const int tiles = max_rows / BM * (N / wide::WBN);
+        gemm_tcgen05_wide_kernel<<<tiles < sm_count ? tiles : sm_count, wide::WTHREADS, wide::W_SMEM_BYTES, stream>>>(map_a, map_w, p);
+        return eg_launch_status();
+    }
     dim3 grid(N / BN, max_rows / BM);
     gemm_tcgen05_kernel<<<grid, THREADS, SMEM_BYTES, stream>>>(map_a, map_w, p);
     return eg_launch_status();
@@ -1039,16 +1064,17 @@ static int gemm_tcgen05_grouped_any(cudaStream_t stream, int epilogue, const voi
 
 // epilogue: 0 store, 2 SwiGLU on interleaved columns, 7 the exact gelu (by erf).
 EG_API int eg_gemm_tcgen05_grouped(cudaStream_t stream, int epilogue, const void* A, long long lda, const void* W, long long ldw, void* out,
-                                   long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, int* status) {
-    return gemm_tcgen05_grouped_any(stream, epilogue, A, lda, W, ldw, out, ldo, max_rows, N, K, groups, tile_group, status, 0.f);
+                                   long long ldo, int max_rows, int N, int K, int groups, const int* tile_group, const int* active_rows,
+                                   int* status) {
+    return gemm_tcgen05_grouped_any(stream, epilogue, A, lda, W, ldw, out, ldo, max_rows, N, K, groups, tile_group, active_rows, status, 0.f);
 }
 
 // The grouped product over interleaved gate and up columns with the clamped gate in its epilogue (out [max_rows, N / 2]):
 // g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(1.702 g) (u + 1).
 EG_API int eg_gemm_tcgen05_grouped_glu(cudaStream_t stream, const void* A, long long lda, const void* W, long long ldw, void* out, long long ldo,
-                                       int max_rows, int N, int K, int groups, const int* tile_group, int* status, float limit) {
+                                       int max_rows, int N, int K, int groups, const int* tile_group, const int* active_rows, int* status, float limit) {
     if (!(limit > 0.f)) return (int)cudaErrorInvalidValue;
-    return gemm_tcgen05_grouped_any(stream, EPI_SWIGLU, A, lda, W, ldw, out, ldo, max_rows, N, K, groups, tile_group, status, limit);
+    return gemm_tcgen05_grouped_any(stream, EPI_SWIGLU, A, lda, W, ldw, out, ldo, max_rows, N, K, groups, tile_group, active_rows, status, limit);
 }
 
 namespace {
