@@ -259,6 +259,54 @@ int main(int argc, char** argv) {
         CHECK(throws<std::invalid_argument>([&] { bad.validate(); }, "names stream addition 3"));
     }
 
+    // ---- a sixth listed design: latent attention in two forms, chunks with slopes and borrowed keys, experts chosen within groups ----
+    {
+        const char* kBorrowed = R"({"architecture": "Mipurax", "vocab": 91, "width": 52, "norm": {"eps": 3e-6},
+          "layers": [
+            {"type": "attention", "mixer": {"heads": 6, "kv_heads": 2, "dim": 12, "vdim": 20, "scale": 0.4, "mask": {"size": 24}}, "mlp": null},
+            {"type": "latent_attention", "mixer": {"heads": 3, "dim": 10, "rot_dim": 6, "vdim": 14, "kv_rank": 22, "q_rank": 18, "scale": 0.3, "rot": {"base": 700, "dims": 6}},
+             "mlp": {"kind": "moe", "router": {"experts": 10, "top": 3, "groups": {"count": 5, "keep": 2}}, "expert": {"ff": 28}, "shared": {"ff": 36}}},
+            {"type": "attention", "mixer": {"heads": 6, "kv_heads": 2, "dim": 12, "vdim": 20, "scale": 0.7, "mask": {"size": 40}, "kv_from": 0}, "mlp": {"kind": "dense", "ff": 44}},
+            {"type": "latent_attention_2", "mixer": {"heads": 1, "dim": 8, "rot_dim": 4, "vdim": 8, "kv_rank": 9, "q_rank": 7, "scale": 1, "rot": {"base": 50.5, "dims": 4}},
+             "mlp": {"kind": "moe", "router": {"experts": 3, "top": 1}, "expert": {"ff": 16}}}]})";
+        const ModelSpec spec = ArchitectureRegistry::instance().build(json::parse(kBorrowed));
+        CHECK(spec.architecture == "mipurax" && spec.layers.size() == 4 && spec.vocab_size == 91 && spec.hidden_size == 52 && spec.run_order.size() == 4);
+        CHECK(spec.run_order[2].layer == 2 && spec.run_order[2].cache == 0 && !spec.run_order[2].writes_cache && spec.run_order[0].writes_cache && spec.run_order[3].cache == 3);
+        const Params &own = spec.layers[0].sublayers[0].part.params, &reader = spec.layers[2].sublayers[0].part.params;
+        CHECK(own.integer("own_keys") == 1 && own.integer("chunk") == 24 && own.integer("cached_back") == 40 && own.integer("slopes") == 1);
+        CHECK(reader.integer("own_keys") == 0 && reader.integer("chunk") == 40 && reader.integer("cached_back") == 40 && reader.real("scale") == 0.7);
+        const Params &first = spec.layers[1].sublayers[0].part.params, &second = spec.layers[3].sublayers[0].part.params;
+        CHECK(first.text("rot_layout") == "interleaved" && first.text("gate") == "values" && !first.flag("sink", true) && first.real("rot_base") == 700.0 && first.integer("rot_dims") == 6);
+        CHECK(second.text("rot_layout") == "half" && second.text("gate") == "heads" && second.flag("sink", false) && second.real("rot_base") == 50.5 && second.real("eps") == 3e-6);
+        const Params &routed = spec.layers[1].sublayers[1].part.params, &plain = spec.layers[3].sublayers[1].part.params;
+        CHECK(routed.integer("groups") == 5 && routed.integer("keep_groups") == 2 && routed.integer("normalize") == 1 && routed.text("activation") == "gelu" &&
+              routed.integer("shared_ff") == 36 && routed.integer("correction") == 0 && routed.text("scoring") == "sigmoid");
+        CHECK(!plain.has("groups") && !plain.has("shared_ff") && spec.layers[0].sublayers.size() == 1 && spec.layers[2].sublayers[1].part.kind == "gelu");
+        CHECK(spec.embedding.params.text("norm_name") == ".norm" && spec.embedding.params.real("norm_offset") == 1.0 && spec.lm_head.params.text("tied_to") == "embed" &&
+              spec.final_norm.params.real("offset") == 1.0);
+        auto changed = [&](const std::string& from, const std::string& to) {
+            std::string text = kBorrowed;
+            const size_t at = text.find(from);
+            CHECK(at != std::string::npos);
+            text.replace(at, from.size(), to);
+            return text;
+        };
+        const ModelSpec open = ArchitectureRegistry::instance().build(json::parse(changed(R"(, "mask": {"size": 40}, "kv_from")", R"(, "kv_from")")));
+        CHECK(open.layers[0].sublayers[0].part.params.integer("cached_back") == -1 && !open.layers[2].sublayers[0].part.params.has("chunk"));
+        for (const auto& wrong : {changed(R"("kv_from": 0)", R"("kv_from": 2)"), changed(R"("kv_from": 0)", R"("kv_from": 1)"), changed(R"("dim": 12, "vdim": 20, "scale": 0.7)", R"("dim": 14, "vdim": 20, "scale": 0.7)"),
+                                  changed(R"("count": 5)", R"("count": 4)"), changed(R"("keep": 2)", R"("keep": 6)"), changed(R"("keep": 2)", R"("keep": 1)"),
+                                  changed(R"("dims": 6)", R"("dims": 5)"), changed(R"("type": "latent_attention_2")", R"("type": "latent")"), changed(R"("size": 24)", R"("size": 0)"),
+                                  changed(R"("kind": "dense")", R"("kind": "gated")"), changed(R"("kv_heads": 2)", R"("kv_heads": 4)")}) {
+            bool refused = false;
+            try {
+                ArchitectureRegistry::instance().build(json::parse(wrong));
+            } catch (const std::exception&) {
+                refused = true;
+            }
+            CHECK(refused);
+        }
+    }
+
     // ---- a fifth listed design: norms in groups, waves of the position, two mixers side by side whose outputs are normed, a delta rule ----
     {
         const char* kFading = R"({"architecture": "Zodosun", "vocab": 83, "width": 60, "norm": {"eps": 2e-6, "groups": 3}, "logit_scale": 1.75,

@@ -84,6 +84,8 @@ ALONE = {
     "latent_2_tensor": model([(latent(2, heads=18, dim=32, rot_dim=16, vdim=40, kv_rank=72, q_rank=40, scale=0.14), None)], width=128),
     "latent_large": model([(latent(1, heads=2, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=64, scale=0.07), None)]),
     "latent_2_large": model([(latent(2, heads=17, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=64, scale=0.07), None)]),
+    "latent_one_head": model([(latent(1, heads=1, dim=16, rot_dim=8, vdim=16, kv_rank=32, q_rank=24, scale=0.2), None),
+                              (latent(2, heads=1, dim=8, rot_dim=16, vdim=8, kv_rank=24, q_rank=16, scale=0.2), None)]),
     "latent_uneven": model([(latent(1, heads=3, dim=5, rot_dim=6, vdim=7, kv_rank=9, q_rank=11, scale=0.4), None)]),
     "chunked": model([(chunked(), None)]),
     "chunked_all_keys": model([(chunked(size=None), None)]),
@@ -97,6 +99,10 @@ ALONE = {
     "another_layers_keys_planes": model([(chunked(heads=4, kv_heads=2, dim=64, vdim=64, scale=0.12, size=50), None),
                                          (chunked(heads=4, kv_heads=2, dim=64, vdim=64, scale=0.2, size=20, kv_from=0), None),
                                          (chunked(heads=4, kv_heads=2, dim=64, vdim=64, scale=0.1, size=None, kv_from=0), None)], width=128),
+    # a width that is no multiple of four, sizes that are no multiples of four either
+    "odd_width": model([(latent(heads=3, dim=10, rot_dim=2, vdim=6, kv_rank=14, q_rank=18, scale=0.3), moe(experts=6, top=2, ff=22, groups=(2, 1), shared=18)),
+                        (chunked(heads=3, kv_heads=1, dim=10, vdim=6, scale=0.4, size=9), 27), (latent(2, heads=2, dim=6, rot_dim=6, vdim=10, kv_rank=10, q_rank=6, scale=0.3), None)],
+                       width=90, vocab=53),
     "dense": model([(chunked(heads=2, kv_heads=2, dim=8, vdim=8), 100)]),
     "routed": model([(chunked(heads=2, kv_heads=1, dim=8, vdim=8), moe())]),
     "routed_no_groups": model([(chunked(heads=2, kv_heads=1, dim=8, vdim=8), moe(experts=7, top=3, groups=None, shared=None))]),
@@ -233,7 +239,7 @@ def test_the_restatements_own_pieces():
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name", ["general", "tensor", "odd", "ones", "latent_tensor", "latent_2_tensor", "latent_large", "latent_2_large", "latent_uneven", "chunked_planes_32",
+@pytest.mark.parametrize("name", ["general", "tensor", "odd", "ones", "latent_tensor", "latent_2_tensor", "latent_large", "latent_2_large", "latent_uneven", "latent_one_head", "odd_width", "chunked_planes_32",
                                   "chunked_planes_64", "chunked_planes_128", "chunked_planes_all_keys", "chunked_large_values", "another_layers_keys",
                                   "another_layers_keys_planes", "routed_grouped_product", "routed_single_members"])
 def test_prompt_whole_and_token_by_token(folders, name, dtype):
