@@ -148,7 +148,20 @@ __global__ void __launch_bounds__(128) moe_select_kernel(const float* __restrict
     const int per = outputs / groups;
     float* group = logit + outputs;
     if (groups > 1) {
-        for (int g = lane; g < groups; g += 32) {
+        const bool in_step = per <= 32 && (per & (per - 1)) == 0;
+        if (in_step) {                           // a lane per output: the two largest of a run by halving
+            for (int e0 = 0; e0 < outputs; e0 += 32) {
+                const int e = e0 + lane;
+                float first = e < outputs ? logit[e] + (correction ? correction[e] : 0.f) : -INFINITY, second = -INFINITY;
+                for (int o = 1; o < per; o <<= 1) {
+                    const float of = __shfl_xor_sync(0xffffffffu, first, o), os = __shfl_xor_sync(0xffffffffu, second, o);
+                    second = fmaxf(fminf(first, of), fmaxf(second, os));
+                    first = fmaxf(first, of);
+                }
+                if (e < outputs && (lane & (per - 1)) == 0) group[e / per] = per > 1 ? first + second : first;
+            }
+        }
+        for (int g = lane; !in_step && g < groups; g += 32) {
             float first = -INFINITY, second = -INFINITY;
             for (int e = g * per; e < (g + 1) * per; ++e) {
                 const float v = logit[e] + (correction ? correction[e] : 0.f);
@@ -169,14 +182,17 @@ __global__ void __launch_bounds__(128) moe_select_kernel(const float* __restrict
         for (int g = lane, i = 0; g < groups; g += 32, ++i) group[g] = (kept >> i) & 1ull ? 1.f : 0.f;
         __syncwarp();
     }
-    float sum_chosen = 0.f;
+    float sum_chosen = 0.f, my_weight = 0.f;
+    int my_id = 0;
     unsigned long long taken = 0ull;             // a lane tracks which of its own outputs are taken: bit k for e = lane + 32 k
+    if (groups > 1)                              // outputs of the groups that are left out count as taken
+        for (int e = lane, i = 0; e < outputs; e += 32, ++i)
+            if (group[e / per] == 0.f) taken |= 1ull << i;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int arg = 0x7fffffff;
         for (int e = lane, i = 0; e < outputs; e += 32, ++i) {
             if ((taken >> i) & 1ull) continue;
-            if (groups > 1 && group[e / per] == 0.f) continue;
             const float v = logit[e] + (correction ? correction[e] : 0.f);
             if (v > best) { best = v; arg = e; }
         }
@@ -186,15 +202,25 @@ __global__ void __launch_bounds__(128) moe_select_kernel(const float* __restrict
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
         if (arg != 0x7fffffff && arg % 32 == lane) taken |= 1ull << (arg / 32);
-        if (lane == 0) {
-            const float s = arg == 0x7fffffff ? 0.f : logit[arg];
-            ids[(size_t)t * top + k] = arg == 0x7fffffff ? outputs : arg;
-            weights[(size_t)t * top + k] = s;
-            sum_chosen += s;
+        // choice k stays with lane k % 32 until 32 of them are written together; the sum is every lane's (the scores lie in shared memory)
+        const float s = arg == 0x7fffffff ? 0.f : logit[arg];
+        sum_chosen += s;
+        if (k % 32 == lane) {
+            my_id = arg == 0x7fffffff ? outputs : arg;
+            my_weight = s;
+        }
+        if (k % 32 == 31 || k == top - 1) {
+            const int at = k / 32 * 32 + lane;
+            if (at <= k) {
+                ids[(size_t)t * top + at] = my_id;
+                weights[(size_t)t * top + at] = normalize && top <= 32 ? my_weight / (sum_chosen + 1e-20f) : my_weight;
+            }
         }
     }
-    if (normalize && lane == 0)
-        for (int k = 0; k < top; ++k) weights[(size_t)t * top + k] /= sum_chosen + 1e-20f;
+    if (normalize && top > 32) {
+        __syncwarp();
+        for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] /= sum_chosen + 1e-20f;       // each lane what it wrote itself
+    }
 }
 
 // grid (token, choice, chunk of ff); a warp per hidden unit; GU [experts, 2 ff, width] with the gate row of unit f at

@@ -209,7 +209,8 @@ def test_each_mechanism_alone(folders, name, dtype):
 
 def test_routers_with_plain_random_weights(tmp_path):
     """The choice itself in 32-bit, from router weights without any order in them: several group layouts."""
-    for i, (experts, top, groups) in enumerate([(12, 3, (4, 2)), (40, 6, (8, 3)), (9, 2, (3, 1)), (66, 4, None), (64, 5, (32, 9)), (70, 7, (70, 20))]):
+    for i, (experts, top, groups) in enumerate([(12, 3, (4, 2)), (40, 6, (8, 3)), (9, 2, (3, 1)), (66, 4, None), (64, 5, (32, 9)), (70, 7, (70, 20)), (32, 4, (8, 3)), (48, 6, (6, 3)),
+                                               (80, 34, (5, 4)), (64, 6, (2, 1))]):
         cfg = model([(chunked(heads=2, kv_heads=1, dim=8, vdim=8), moe(experts=experts, top=top, groups=groups, ff=16, shared=None))])
         w = pm.random_weights(cfg, 30 + i)
         folder = pm.write_model_dir(tmp_path / str(i), cfg, w)
